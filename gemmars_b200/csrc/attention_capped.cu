@@ -16,7 +16,8 @@
 //                          keys 0..keep_first-1 as well, wherever the window stands; softmax, whose
 //                          denominator also holds exp(sink[head]) when sinks are given (a term
 //                          without key or value); output times sigmoid(gate) * out_scale when a
-//                          gate is given
+//                          gate is given (a number per output channel, or with gate_per_head one
+//                          per head)
 //
 // Cache layout as everywhere in the package: keys [pages, kv_heads, page_size, D], values
 // transposed inside a page [pages, kv_heads, Vd, page_size].
@@ -152,7 +153,7 @@ __global__ void __launch_bounds__(CHUNK) attention_capped_kernel(
     const T* __restrict__ vcache, const int* __restrict__ page_table, int table_width, int page_size, int G, int D, int Vd,
     const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ seq_slot, int H, int window,
     int keep_first, const float* __restrict__ sink, float scale, float cap, const T* __restrict__ gate, long long gate_stride,
-    float out_scale) {
+    float out_scale, int gate_per_head) {
   extern __shared__ float smem[];
   pdl_release_next();
   pdl_wait_prior();
@@ -213,7 +214,7 @@ __global__ void __launch_bounds__(CHUNK) attention_capped_kernel(
     const int d = tid + u * CHUNK;
     if (d < Vd) {
       float o = acc[u] / l;
-      if (gate) o *= 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * gate_stride + (size_t)h * Vd + d])));
+      if (gate) o *= 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * gate_stride + (gate_per_head ? h : h * Vd + d)])));
       orow[d] = from_f32<T>(o * out_scale);
     }
   }
@@ -223,7 +224,8 @@ GB_EXPORT int gb_attention_capped(const void* q, long long q_stride, void* out, 
                                   const void* kcache, const void* vcache, const int* page_table, int table_width, int page_size,
                                   int G, int D, int Vd, const int* tok_pos, const int* tok_seq, const int* seq_slot, int ntok,
                                   int H, int window, int keep_first, const float* sink, float scale, float cap,
-                                  const void* gate, long long gate_stride, float out_scale, cudaStream_t stream) {
+                                  const void* gate, long long gate_stride, float out_scale, int gate_per_head,
+                                  cudaStream_t stream) {
   if (ntok <= 0) return 0;
   if (D <= 0 || Vd <= 0 || Vd > VPT * CHUNK || G <= 0 || H % G || keep_first < 0) return GB_ERR_SIZE;
   if (window <= 0) keep_first = 0;      // every key is seen already
@@ -232,11 +234,11 @@ GB_EXPORT int gb_attention_capped(const void* q, long long q_stride, void* out, 
   if (dtype == GB_F32)
     gb_launch(attention_capped_kernel<float>, grid, CHUNK, smem, stream, (const float*)q, q_stride, (float*)out, out_stride,
               (const float*)kcache, (const float*)vcache, page_table, table_width, page_size, G, D, Vd, tok_pos, tok_seq,
-              seq_slot, H, window, keep_first, sink, scale, cap, (const float*)gate, gate_stride, out_scale);
+              seq_slot, H, window, keep_first, sink, scale, cap, (const float*)gate, gate_stride, out_scale, gate_per_head);
   else if (dtype == GB_BF16)
     gb_launch(attention_capped_kernel<bf16>, grid, CHUNK, smem, stream, (const bf16*)q, q_stride, (bf16*)out, out_stride,
               (const bf16*)kcache, (const bf16*)vcache, page_table, table_width, page_size, G, D, Vd, tok_pos, tok_seq, seq_slot,
-              H, window, keep_first, sink, scale, cap, (const bf16*)gate, gate_stride, out_scale);
+              H, window, keep_first, sink, scale, cap, (const bf16*)gate, gate_stride, out_scale, gate_per_head);
   else
     return GB_ERR_DTYPE;
   return gb_launch_status();

@@ -3,7 +3,8 @@
 // pair of sizes), score = (q . k) * scale, then cap * tanh(score / cap) when cap > 0, a window when
 // given (with `keep_first`, the keys 0..keep_first-1 are seen wherever the window stands), a sink
 // per head when given (exp(sink[head]) joins the softmax's denominator, with no key and no value),
-// and the output times sigmoid(gate) * out_scale when a gate is given.
+// and the output times sigmoid(gate) * out_scale when a gate is given (a number per output channel, or
+// with gate_per_head one per head).
 //
 // The arrangement is that of attention_prefill.cu: the 16 rows of an MMA are 16 consecutive
 // tokens of one sequence for one query head, each row masked at its own position and window;
@@ -47,7 +48,8 @@ attention_capped_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16
                          const int* __restrict__ cu_seqlens, const int* __restrict__ seq_start,
                          const int* __restrict__ seq_slot, int n_seqs, int nh, int window, int keep_first,
                          const float* __restrict__ sink, int heads_per_cta, float scale,
-                         float cap, const bf16* __restrict__ gate, long long gate_stride, float out_scale) {
+                         float cap, const bf16* __restrict__ gate, long long gate_stride, float out_scale,
+                         int gate_per_head) {
   pdl_release_next();
   pdl_wait_prior();
   // ---- which sequence and which 64-token tile of it
@@ -181,9 +183,11 @@ attention_capped_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16
     l1 = l1 * keep1 + exp2f(s2 - n1);
   }
   if (v0) {
-    const float inv = out_scale * keep0 / l0;
+    float inv = out_scale * keep0 / l0;
+    if (gate && gate_per_head)
+      inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)(tok0 + g) * gate_stride + head])));
     bf16* dst = out + (size_t)(tok0 + g) * out_stride + (size_t)head * VD + 2 * c;
-    const bf16* gt = gate ? gate + (size_t)(tok0 + g) * gate_stride + (size_t)head * VD + 2 * c : nullptr;
+    const bf16* gt = gate && !gate_per_head ? gate + (size_t)(tok0 + g) * gate_stride + (size_t)head * VD + 2 * c : nullptr;
 #pragma unroll
     for (int d = 0; d < VD / 8; ++d) {
       float a = o[d][0] * inv, bb = o[d][1] * inv;
@@ -196,9 +200,11 @@ attention_capped_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16
     }
   }
   if (v1) {
-    const float inv = out_scale * keep1 / l1;
+    float inv = out_scale * keep1 / l1;
+    if (gate && gate_per_head)
+      inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)(tok0 + g + 8) * gate_stride + head])));
     bf16* dst = out + (size_t)(tok0 + g + 8) * out_stride + (size_t)head * VD + 2 * c;
-    const bf16* gt = gate ? gate + (size_t)(tok0 + g + 8) * gate_stride + (size_t)head * VD + 2 * c : nullptr;
+    const bf16* gt = gate && !gate_per_head ? gate + (size_t)(tok0 + g + 8) * gate_stride + (size_t)head * VD + 2 * c : nullptr;
 #pragma unroll
     for (int d = 0; d < VD / 8; ++d) {
       float a = o[d][2] * inv, bb = o[d][3] * inv;
@@ -223,7 +229,8 @@ attention_capped_single_kernel(const bf16* __restrict__ q, long long q_stride, b
                          const int* __restrict__ cu_seqlens, const int* __restrict__ seq_start,
                          const int* __restrict__ seq_slot, int n_seqs, int nh, int window, int keep_first,
                          const float* __restrict__ sink, float scale,
-                         float cap, const bf16* __restrict__ gate, long long gate_stride, float out_scale) {
+                         float cap, const bf16* __restrict__ gate, long long gate_stride, float out_scale,
+                         int gate_per_head) {
   pdl_release_next();
   pdl_wait_prior();
   const int b = blockIdx.x;
@@ -365,7 +372,7 @@ attention_capped_single_kernel(const bf16* __restrict__ q, long long q_stride, b
     }
     float a = acc * out_scale / total;
     const size_t at = (size_t)(head_base + row) * VD + col;
-    if (gate) a *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)tok0 * gate_stride + at])));
+    if (gate) a *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)tok0 * gate_stride + (gate_per_head ? head_base + row : at)])));
     out[(size_t)tok0 * out_stride + at] = __float2bfloat16_rn(a);
   }
 }
@@ -379,12 +386,13 @@ GB_EXPORT int gb_attention_capped_mma(const void* q, long long q_stride, void* o
                                       const void* kcache, const void* vcache, const int* page_table, int table_width,
                                       int page_size, int nkv, int hd, int vd, const int* cu_seqlens, const int* seq_start,
                                       const int* seq_slot, int n_seqs, int ntok, int nh, int window, int keep_first,
-                                      const float* sink, float scale, float cap, const void* gate, long long gate_stride, float out_scale, int single, cudaStream_t stream) {
+                                      const float* sink, float scale, float cap, const void* gate, long long gate_stride, float out_scale, int gate_per_head,
+                                      int single, cudaStream_t stream) {
   if (ntok <= 0 || n_seqs <= 0) return 0;
   if (hd != HD || vd != VD || nkv <= 0 || nh % nkv || page_size % KEYS || keep_first < 0) return GB_ERR_SIZE;
   if (window <= 0) keep_first = 0;      // every key is seen already
   if (((uintptr_t)q & 15) || (q_stride % 8) || ((uintptr_t)out & 3) || (out_stride % 2) || ((uintptr_t)kcache & 15) ||
-      ((uintptr_t)vcache & 15) || ((uintptr_t)gate & 3) || (gate_stride % 2))
+      ((uintptr_t)vcache & 15) || (!gate_per_head && (((uintptr_t)gate & 3) || (gate_stride % 2))))
     return GB_ERR_SIZE;
   PagedKV kv{page_table, table_width, page_size, nkv, hd};
   const int rep = nh / nkv;
@@ -403,7 +411,7 @@ GB_EXPORT int gb_attention_capped_mma(const void* q, long long q_stride, void* o
     if ((size_t)sgrid.x * sgrid.y > 2 * 148) {
       gb_launch(attention_capped_single_kernel, sgrid, SPLIT * 32, smem, stream,
           (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kcache, (const bf16*)vcache, kv, cu_seqlens,
-          seq_start, seq_slot, n_seqs, nh, window, keep_first, sink, scale, cap, (const bf16*)gate, gate_stride, out_scale);
+          seq_start, seq_slot, n_seqs, nh, window, keep_first, sink, scale, cap, (const bf16*)gate, gate_stride, out_scale, gate_per_head);
     } else {
       // few CTAs: started only when the kernel before has ended, so that they spread one to an SM instead of
       // sharing the few SMs that had room while that kernel ran
@@ -414,13 +422,13 @@ GB_EXPORT int gb_attention_capped_mma(const void* q, long long q_stride, void* o
       cfg.stream = stream;
       cudaLaunchKernelEx(&cfg, attention_capped_single_kernel,
           (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kcache, (const bf16*)vcache, kv, cu_seqlens,
-          seq_start, seq_slot, n_seqs, nh, window, keep_first, sink, scale, cap, (const bf16*)gate, gate_stride, out_scale);
+          seq_start, seq_slot, n_seqs, nh, window, keep_first, sink, scale, cap, (const bf16*)gate, gate_stride, out_scale, gate_per_head);
     }
     return gb_launch_status();
   }
   dim3 grid((ntok + TILE - 1) / TILE + n_seqs, nkv * chunks);
   gb_launch(attention_capped_mma_kernel, grid, MT * heads_per_cta * 32, 0, stream,
       (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kcache, (const bf16*)vcache, kv, cu_seqlens,
-      seq_start, seq_slot, n_seqs, nh, window, keep_first, sink, heads_per_cta, scale, cap, (const bf16*)gate, gate_stride, out_scale);
+      seq_start, seq_slot, n_seqs, nh, window, keep_first, sink, heads_per_cta, scale, cap, (const bf16*)gate, gate_stride, out_scale, gate_per_head);
   return gb_launch_status();
 }

@@ -9,13 +9,15 @@
 #include "common.cuh"
 
 enum { OUT_STORE = 0, OUT_ACCUMULATE_F32 = 1 };
+enum { ACT_NONE = 0, ACT_GELU = 1, ACT_RELU2 = 2 };   // the exact (erf) GELU; the square of relu
 
 constexpr int BM = 64, BN = 64, BK = 16;
 
 template <typename TI, typename TO, int MODE>
 __global__ void __launch_bounds__(256) gemm_ref_kernel(const TI* __restrict__ x, const TI* __restrict__ w,
                                                        const float* __restrict__ bias, TO* __restrict__ y, int M,
-                                                       int N, int K, long long ldx, long long ldy) {
+                                                       int N, int K, long long ldx, long long ldy, int act,
+                                                       const float* __restrict__ col_scale) {
   pdl_release_next();
   pdl_wait_prior();
   __shared__ float xs[BK][BM + 4];
@@ -56,6 +58,9 @@ __global__ void __launch_bounds__(256) gemm_ref_kernel(const TI* __restrict__ x,
       const int gn = n0 + tn + j;
       if (gn >= N) continue;
       float v = acc[i][j] + (bias ? bias[gn] : 0.f);
+      if (act == ACT_GELU) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
+      else if (act == ACT_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
+      if (col_scale) v *= col_scale[gn];
       TO* dst = y + (size_t)gm * ldy + gn;
       if (MODE == OUT_ACCUMULATE_F32)
         *dst = from_f32<TO>(to_f32(*dst) + v);
@@ -66,15 +71,19 @@ __global__ void __launch_bounds__(256) gemm_ref_kernel(const TI* __restrict__ x,
 }
 
 // x: [M, K] rows ldx apart; w: [N, K]; y: [M, N] rows ldy apart.
-// mode OUT_STORE writes y in out_dtype; OUT_ACCUMULATE_F32 adds into a float32 y.
+// mode OUT_STORE writes y in out_dtype; OUT_ACCUMULATE_F32 adds into a float32 y.  act: an activation of
+// product + bias; col_scale (null: ones): [N], multiplied in after it, before the store or the add.
 GB_EXPORT int gb_gemm_ref(const void* x, const void* w, int in_dtype, const float* bias, void* y, int out_dtype,
-                          int mode, int M, int N, int K, long long ldx, long long ldy, cudaStream_t stream) {
+                          int mode, int M, int N, int K, long long ldx, long long ldy, int act, const float* col_scale,
+                          cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0) return GB_ERR_SIZE;
+  if (act < ACT_NONE || act > ACT_RELU2) return GB_ERR_ARG;
   dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
   if (mode == OUT_ACCUMULATE_F32 && out_dtype != GB_F32) return GB_ERR_DTYPE;
 #define LAUNCH(TI, TO, MODE) \
-  gb_launch(gemm_ref_kernel<TI, TO, MODE>, grid, 256, 0, stream, (const TI*)x, (const TI*)w, bias, (TO*)y, M, N, K, ldx, ldy)
+  gb_launch(gemm_ref_kernel<TI, TO, MODE>, grid, 256, 0, stream, (const TI*)x, (const TI*)w, bias, (TO*)y, M, N, K, ldx, ldy, \
+            act, col_scale)
   if (in_dtype == GB_F32) {
     if (out_dtype != GB_F32) return GB_ERR_DTYPE;
     if (mode == OUT_ACCUMULATE_F32) LAUNCH(float, float, OUT_ACCUMULATE_F32);

@@ -77,6 +77,8 @@ struct QkvTail {
   const float2* rope_table; // prompts: [tokens][64] (cos, sin) of each packed token's angles, or null
   const int2* token_place;  // prompts: [tokens] (page, position in the page) of each packed token
   NormLink link;            // any mode of gemm_tc_kernel: a norm taken into this product (all null: none)
+  const float* col_scale;   // EPI_ACCUMULATE_F32: [N], y += col_scale[n] * (product + bias); null: one
+  int act;                  // EPI_STORE_BF16: an activation of (product + bias) before the rounding (see out_act)
   int recv_apart;           // gemm_tc_kernel with a split inner dimension: the ranks' partial sums arrive in
                             // memory of their own behind the stages (see the exchange), not in the stages
 };
@@ -104,6 +106,16 @@ __device__ __forceinline__ float silu_mul(float g, float u) {
 #else
 __device__ __forceinline__ float silu_mul(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
 #endif
+
+// Activations of a product without a gate: 1 the exact (erf) GELU, 2 the square of relu.
+enum { OUT_ACT_NONE = 0, OUT_ACT_GELU = 1, OUT_ACT_RELU2 = 2 };
+__device__ __forceinline__ float out_act(float x, int act) {
+  if (act == OUT_ACT_RELU2) {
+    const float r = fmaxf(x, 0.f);
+    return r * r;
+  }
+  return act == OUT_ACT_GELU ? 0.5f * x * (1.0f + erff(x * 0.70710678118654752f)) : x;
+}
 
 template <int MODE>
 __device__ __forceinline__ void emit(void* y, size_t idx, float v) {
@@ -198,6 +210,15 @@ __device__ __forceinline__ void store_direct(void* y, long long ldy, const uint3
     for (int j = 0; j < 16; ++j)
       if (m_first + j < M) emit<MODE>(y, (size_t)(m_first + j) * ldy + n, __uint_as_float(v[j]) + bias);
   }
+}
+
+__device__ __forceinline__ void scale_values(uint32_t (&v)[16], float s) {
+#pragma unroll
+  for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) * s);
+}
+__device__ __forceinline__ void act_values(uint32_t (&v)[16], float bias, int act) {
+#pragma unroll
+  for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(out_act(__uint_as_float(v[j]) + bias, act));
 }
 
 // The accumulator columns [c, c + 16) of this warp's 32 lanes, gated when the tile has two
@@ -550,13 +571,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 
   // ---------------- epilogue (warps 0-3); the other warps wait at the barriers below
   bool have_acc = false;
-  float bias_v = 0.f, old[8];
+  float bias_v = 0.f, col_v = 1.f, old[8];
   __shared__ float row_scale[64], sq_part[4][32];
   const NormLink& link = tail.link;
   if (warp < 4) {
     pdl_wait_prior();   // y may be read (accumulate) and is written: not before the kernel before is done
     const int n = n0 + warp * 32 + lane;
     bias_v = (bias && n < N) ? bias[n] : 0.f;
+    if (MODE == EPI_ACCUMULATE_F32 && tail.col_scale) {
+      col_v = n < N ? tail.col_scale[n] : 0.f;
+      bias_v *= col_v;
+    }
     if (link.in_partial) {
       // The scale of each of the tile's tokens, while the products run.  A token's sums of squares
       // (one per tile of the product that left them) are shared out over 128 / BN adjacent lanes,
@@ -654,6 +679,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         for (int r = 1; r < 8; ++r) sum += part[r];
         const float sc = link.in_partial ? row_scale[c] : 1.f;
         sum *= sc;
+        if (MODE == EPI_ACCUMULATE_F32) sum *= col_v;
         if (MODE == EPI_QKV_BF16) {   // every thread has the same tokens: they finish one together
           qkv_finish(tail, y, ldy, m0 + c, n0, f, sum + bias_v, qkv_red, qkv_xs);
           continue;
@@ -675,7 +701,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             ((float*)y)[idx] = final_r;
             if (link.out_weight) link.out_rows[(size_t)(m0 + c) * link.out_ld + n] = __float2bfloat16_rn(final_r * out_g);
           } else {
-            emit<MODE>(y, idx, sum + bias_v);
+            emit<MODE>(y, idx, MODE == EPI_STORE_BF16 ? out_act(sum + bias_v, tail.act) : sum + bias_v);
           }
         }
         if (MODE == EPI_ACCUMULATE_F32 && link.out_weight) {   // this warp's 32 features of the token's sum of squares
@@ -692,7 +718,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     }
   } else if (warp < 4 && have_acc) {
     const int f = warp * 32 + lane, n = n0 + f;
-    const float b = bias_v;
+    float b = bias_v;
     // the pipeline's stages are idle by now: the pieces on their way out lie there
     TileOut<MODE> tile_out(&map_y, smem, warp);
     const bool by_tma = MODE != EPI_QKV_BF16 && y_tma != 0;
@@ -717,6 +743,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       }
       gate<DUAL>(v, u);
       if (BOTH) gate<DUAL>(v2, u2);
+      if (MODE == EPI_ACCUMULATE_F32 && tail.col_scale) {
+        scale_values(v, col_v);
+        if (BOTH) scale_values(v2, col_v);
+      }
+      if (MODE == EPI_STORE_BF16 && tail.act) {
+        act_values(v, bias_v, tail.act);
+        if (BOTH) act_values(v2, bias_v, tail.act);
+        b = 0.f;
+      }
       if (by_tma) {
         tile_out.send(v, v2, BOTH, b, lane, n0 + warp * 32, m0 + c, N);
       } else if (MODE == EPI_QKV_BF16) {
@@ -811,8 +846,8 @@ constexpr int PERSISTENT_QKV_THREADS = 320, QKV_STAGING_BYTES = 65 * 1024;   // 
 // group; tile_expert[m tile] names it (-1: a tile no group uses, which every role skips) and the
 // tile's rows of W are the group's (W stacks the groups' matrices, rows_per_expert each).  The gated
 // mode then applies g = min(g, limit), u = clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + shift)
-// when limit > 0, and multiplies row r of the result by row_scale[r].  `act` 1 (bfloat16 results of
-// a product without a gate): the exact (erf) GELU of every result, then the row's scale.
+// when limit > 0, and multiplies row r of the result by row_scale[r].  `act` (bfloat16 results of a
+// product without a gate, grouped or not): an activation of every result (out_act), then the row's scale.
 struct Grouped {
   const int* tile_expert = nullptr;
   const float* row_scale = nullptr;
@@ -820,12 +855,11 @@ struct Grouped {
   float limit = 0.f, alpha = 0.f, shift = 0.f;
   int act = 0;
 };
-__device__ __forceinline__ void gelu_rows(uint32_t (&v)[16], const float* row_scale, int row, int M) {
+__device__ __forceinline__ void act_rows(uint32_t (&v)[16], float bias, int act, const float* row_scale, int row, int M) {
 #pragma unroll
   for (int j = 0; j < 16; ++j) {
-    const float x = __uint_as_float(v[j]);
     const float sc = row_scale ? (row + j < M ? row_scale[row + j] : 0.f) : 1.f;
-    v[j] = __float_as_uint(0.5f * x * (1.0f + erff(x * 0.70710678118654752f)) * sc);
+    v[j] = __float_as_uint(out_act(__uint_as_float(v[j]) + bias, act) * sc);
   }
 }
 __device__ __forceinline__ float clamped_gate(float g, float u, const Grouped& grp) {
@@ -1010,7 +1044,12 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
       }
       if (!have) break;
       tc_fence_after();
-      const float bv = (bias && n < N && w.kb0 == 0) ? bias[n] : 0.f;
+      float bv = (bias && n < N && w.kb0 == 0) ? bias[n] : 0.f;
+      float col_v = 1.f;
+      if (MODE == EPI_ACCUMULATE_F32 && tail.col_scale) {
+        col_v = n < N ? tail.col_scale[n] : 0.f;
+        bv *= col_v;
+      }
       // The parts of a tile are added in their order along the inner dimension, so that the sums
       // have the same bits every run: a word per tile and warp counts the parts whose sums are in
       // memory, part q adds when it reads q (its predecessors were walked earlier, or at the same
@@ -1077,15 +1116,21 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
           }
           qkv_prompt_round<MODE, SLOT>(tail, x, n0 / BM, quarter, lane, m0 + c, M, tail.nh * BM, tail_shared, tile_out, 1 + group);
         } else {
-          if (MODE == EPI_STORE_BF16 && grp.act == 1) {
-            gelu_rows(v, grp.row_scale, m0 + c, M);
-            if (both) gelu_rows(v2, grp.row_scale, m0 + c + 16, M);
+          float b_out = bv;
+          if (MODE == EPI_STORE_BF16 && grp.act) {
+            act_rows(v, bv, grp.act, grp.row_scale, m0 + c, M);
+            if (both) act_rows(v2, bv, grp.act, grp.row_scale, m0 + c + 16, M);
+            b_out = 0.f;
+          }
+          if (MODE == EPI_ACCUMULATE_F32 && tail.col_scale) {
+            scale_values(v, col_v);
+            if (both) scale_values(v2, col_v);
           }
           if (y_tma) {
-            tile_out.send(v, v2, both, bv, lane, n0 + warp * 32, m0 + c, N);
+            tile_out.send(v, v2, both, b_out, lane, n0 + warp * 32, m0 + c, N);
           } else {
-            store_direct<MODE>(y, ldy, v, bv, m0 + c, M, n, N);
-            if (both) store_direct<MODE>(y, ldy, v2, bv, m0 + c + 16, M, n, N);
+            store_direct<MODE>(y, ldy, v, b_out, m0 + c, M, n, N);
+            if (both) store_direct<MODE>(y, ldy, v2, b_out, m0 + c + 16, M, n, N);
           }
         }
       }
@@ -1275,10 +1320,14 @@ int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mx, const OutMap
 // Needs K % 8 == 0, ldx % 8 == 0 and 16-byte aligned x and w (TMA rules).
 static int gemm_tc_with_link(const void* x, const void* w, const float* bias, void* y, int mode, int M, int N, int K,
                              long long ldx, long long ldy, int bn, int splits, int stages, const NormLink& link,
-                             cudaStream_t stream) {
+                             int act, const float* col_scale, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
+  if (act < OUT_ACT_NONE || act > OUT_ACT_RELU2 || (act && mode != EPI_STORE_BF16)) return GB_ERR_ARG;
+  if (col_scale && mode != EPI_ACCUMULATE_F32) return GB_ERR_ARG;
   QkvTail tail{};
   tail.link = link;
+  tail.act = act;
+  tail.col_scale = col_scale;
   if (link.in_partial && (M > 64 || bn > 64 || link.in_tiles <= 0)) return GB_ERR_SIZE;
   // leaving rows for a norm is the work of the ranks that finish a token: it needs the inner dimension split
   if (link.out_weight && (mode != EPI_ACCUMULATE_F32 || splits < 2 || M > 64 || !link.out_rows || !link.out_partial)) return GB_ERR_ARG;
@@ -1323,7 +1372,7 @@ static int gemm_tc_with_link(const void* x, const void* w, const float* bias, vo
 
 GB_EXPORT int gb_gemm_tc(const void* x, const void* w, const float* bias, void* y, int mode, int M, int N, int K,
                          long long ldx, long long ldy, int bn, int splits, int stages, cudaStream_t stream) {
-  return gemm_tc_with_link(x, w, bias, y, mode, M, N, K, ldx, ldy, bn, splits, stages, NormLink{}, stream);
+  return gemm_tc_with_link(x, w, bias, y, mode, M, N, K, ldx, ldy, bn, splits, stages, NormLink{}, OUT_ACT_NONE, nullptr, stream);
 }
 
 // gb_gemm_tc with an RMSNorm taken into it (see NormLink; at most 64 tokens).  in_partial non-null:
@@ -1331,13 +1380,16 @@ GB_EXPORT int gb_gemm_tc(const void* x, const void* w, const float* bias, void* 
 // 1 / sqrt(sum of in_partial[0 .. in_tiles)[token] / in_width + in_eps).  out_weight non-null
 // (mode 2, splits >= 2): besides adding into y, the kernel writes bf16(y * out_weight) to out_rows
 // (rows out_ld apart) and this product's tiles' sums of squares to out_partial [ceil(N / 128)][64].
+// act (mode 0): 1 the exact GELU, 2 the square of relu of every result.  col_scale (mode 2; null: ones):
+// [N], y += col_scale * (x w^T + bias).  Both also without a norm.
 GB_EXPORT int gb_gemm_tc_linked(const void* x, const void* w, const float* bias, void* y, int mode, int M, int N, int K,
                                 long long ldx, long long ldy, int bn, int splits, int stages, const float* in_partial,
                                 int in_tiles, float in_eps, int in_width, const float* out_weight, void* out_rows,
-                                long long out_ld, float* out_partial, cudaStream_t stream) {
+                                long long out_ld, float* out_partial, int act, const float* col_scale,
+                                cudaStream_t stream) {
   NormLink link{in_partial, in_tiles, in_eps, in_width > 0 ? 1.0f / (float)in_width : 0.f, out_weight, (bf16*)out_rows, out_ld,
                 out_partial};
-  return gemm_tc_with_link(x, w, bias, y, mode, M, N, K, ldx, ldy, bn, splits, stages, link, stream);
+  return gemm_tc_with_link(x, w, bias, y, mode, M, N, K, ldx, ldy, bn, splits, stages, link, act, col_scale, stream);
 }
 
 // The q/k/v product of a decode step with the per-head work in its epilogue (head size 128, at most
@@ -1380,11 +1432,17 @@ GB_EXPORT int gb_gemm_tc_qkv(const void* x, const void* w, const float* bias, vo
 // 256; ctas: CTAs to launch.  part_flags: null, or 4 * ctas int32 zeros: a product that adds into y
 // may then cut the tiles of a last round that is not full into parts along the inner dimension;
 // every launch leaves the words zero, and two launches that use the same words must not run at
-// the same time.
+// the same time.  act, col_scale: as gb_gemm_tc_linked.
 GB_EXPORT int gb_gemm_tc_persistent(const void* x, const void* w, const float* bias, void* y, int mode, int M, int N,
-                                    int K, long long ldx, long long ldy, int bn, int ctas, int* part_flags,
-                                    cudaStream_t stream) {
+                                    int K, long long ldx, long long ldy, int bn, int ctas, int* part_flags, int act,
+                                    const float* col_scale, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
+  if (act < OUT_ACT_NONE || act > OUT_ACT_RELU2 || (act && mode != EPI_STORE_BF16)) return GB_ERR_ARG;
+  if (col_scale && mode != EPI_ACCUMULATE_F32) return GB_ERR_ARG;
+  QkvTail tail{};
+  tail.col_scale = col_scale;
+  Grouped grp;
+  grp.act = act;
   if (K <= 0 || (K % 8) || (ldx % 8) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ctas <= 0) return GB_ERR_SIZE;
   if (bn < 16 || bn > 256 || (bn % 16)) return GB_ERR_SIZE;
   const bool swiglu = mode == EPI_SWIGLU_BF16;
@@ -1400,17 +1458,17 @@ GB_EXPORT int gb_gemm_tc_persistent(const void* x, const void* w, const float* b
   }
   if (bn > 128) {
     switch (mode) {
-      case EPI_STORE_BF16: return launch_persistent<256, 4, EPI_STORE_BF16>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream);
+      case EPI_STORE_BF16: return launch_persistent<256, 4, EPI_STORE_BF16>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream, tail, nullptr, grp);
       case EPI_STORE_F32: return launch_persistent<256, 4, EPI_STORE_F32>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream);
       case EPI_ACCUMULATE_F32:
-        return launch_persistent<256, 4, EPI_ACCUMULATE_F32>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream, QkvTail{}, part_flags);
+        return launch_persistent<256, 4, EPI_ACCUMULATE_F32>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream, tail, part_flags);
     }
   } else {
     switch (mode) {
-      case EPI_STORE_BF16: return launch_persistent<128, 6, EPI_STORE_BF16>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream);
+      case EPI_STORE_BF16: return launch_persistent<128, 6, EPI_STORE_BF16>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream, tail, nullptr, grp);
       case EPI_STORE_F32: return launch_persistent<128, 6, EPI_STORE_F32>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream);
       case EPI_ACCUMULATE_F32:
-        return launch_persistent<128, 6, EPI_ACCUMULATE_F32>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream, QkvTail{}, part_flags);
+        return launch_persistent<128, 6, EPI_ACCUMULATE_F32>(mw, mx, my, bias, y, M, N, K, ldy, bn, ctas, stream, tail, part_flags);
     }
   }
   return GB_ERR_ARG;
@@ -1420,12 +1478,13 @@ GB_EXPORT int gb_gemm_tc_persistent(const void* x, const void* w, const float* b
 // group after the other, each group starting at a multiple of bn rows (M counts the padding);
 // w stacks `experts` matrices of N rows (2 N gated: gate rows, then up rows); tile_expert [M / bn].
 // mode 1: y float32 [M, N] = x W_g^T; mode 3: y bfloat16 [M, N] = row_scale * act(gate, up), act the
-// clamped form when limit > 0; mode 0: y bfloat16 [M, N] = row_scale * gelu(x W_g^T) (erf form; no
-// gate rows in w).  bn: 128 or 256.
+// clamped form when limit > 0; mode 0: y bfloat16 [M, N] = row_scale * act(x W_g^T) (no gate rows in w;
+// act 1: the exact GELU, 2: the square of relu).  bn: 128 or 256.
 GB_EXPORT int gb_gemm_tc_grouped(const void* x, const void* w, void* y, int mode, int M, int N, int K, long long ldx,
                                  long long ldy, int bn, int ctas, int experts, const int* tile_expert, const float* row_scale,
-                                 float limit, float alpha, float shift, cudaStream_t stream) {
+                                 float limit, float alpha, float shift, int act, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || experts <= 0) return 0;
+  if (act < OUT_ACT_NONE || act > OUT_ACT_RELU2) return GB_ERR_ARG;
   if (K <= 0 || (K % 8) || (ldx % 8) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ctas <= 0) return GB_ERR_SIZE;
   if ((bn != 128 && bn != 256) || M % bn || !tile_expert) return GB_ERR_SIZE;
   const bool gated = mode == EPI_SWIGLU_BF16;
@@ -1435,7 +1494,7 @@ GB_EXPORT int gb_gemm_tc_grouped(const void* x, const void* w, void* y, int mode
   grp.row_scale = (gated || mode == EPI_STORE_BF16) ? row_scale : nullptr;
   grp.rows_per_expert = N * (gated ? 2 : 1);
   grp.limit = limit; grp.alpha = alpha; grp.shift = shift;
-  grp.act = mode == EPI_STORE_BF16 ? 1 : 0;
+  grp.act = mode == EPI_STORE_BF16 ? act : OUT_ACT_NONE;
   CUtensorMap mw, mx;
   if (!tensor_map(&mw, w, (uint64_t)experts * grp.rows_per_expert, (uint64_t)K, (uint64_t)K * 2, gated ? BM / 2 : BM)) return GB_ERR_ARG;
   if (!tensor_map(&mx, x, (uint64_t)M, (uint64_t)K, (uint64_t)ldx * 2, (uint32_t)bn)) return GB_ERR_ARG;

@@ -34,9 +34,12 @@ struct GroupedArgs {
   const int* offsets;                        // [groups + 1], or null: every group has `rows` rows
   int groups, rows, N, K;
   float limit, alpha, shift;                 // gated: g = min(g, limit), u = clamp(u, +-limit), g * sigmoid(alpha g) * (u + shift)
-  int act;                                   // plain mode: 1 = the exact (erf) GELU of every result before the scale
+  int act;                                   // plain mode: an activation of every result before the scale (plain_act)
 };
-__device__ __forceinline__ float gelu_erf_f(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f)); }
+__device__ __forceinline__ float plain_act(float x, int act) {    // 1: the exact (erf) GELU; 2: the square of relu
+  if (act == 2) return fmaxf(x, 0.f) * fmaxf(x, 0.f);
+  return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f));
+}
 
 __device__ __forceinline__ void cp_async16_or_zero(void* smem, const void* gmem, bool valid) {
   const uint32_t s = (uint32_t)__cvta_generic_to_shared(smem);
@@ -180,7 +183,7 @@ __global__ void __launch_bounds__(256, 2) grouped_gemm_kernel(GroupedArgs p) {
         for (int j = 0; j < 4; ++j) {
           const int col = n0 + wn * 32 + j * 8 + 2 * cq;
           float x = acc[i][j][2 * half], y = acc[i][j][2 * half + 1];
-          if (p.act == 1) { x = gelu_erf_f(x); y = gelu_erf_f(y); }
+          if (p.act) { x = plain_act(x, p.act); y = plain_act(y, p.act); }
           x *= sc; y *= sc;
           if (col + 1 < p.N && ((uintptr_t)(dst + col) & (2 * sizeof(TO) - 1)) == 0) {
             store2(dst + col, x, y);
@@ -276,16 +279,18 @@ __global__ void __launch_bounds__(128) moe_permute_kernel(const bf16* __restrict
   if (threadIdx.x == 0) scale[r] = wts[e];
 }
 
-// residual[t] += sum over the token's slots, in slot order, of the rows the down product left
+// residual[t] += col_scale (null: ones) * the sum over the token's slots, in slot order, of the rows the
+// down product left
 __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ place,
-                                                          float* __restrict__ residual, long long ldr, int width, int top) {
+                                                          float* __restrict__ residual, long long ldr, int width, int top,
+                                                          const float* __restrict__ col_scale) {
   pdl_release_next();
   pdl_wait_prior();
   const int t = blockIdx.x;
   for (int n = threadIdx.x; n < width; n += 256) {
     float total = 0.f;
     for (int k = 0; k < top; ++k) total += rows[(size_t)place[(size_t)t * top + k] * width + n];
-    residual[(size_t)t * ldr + n] += total;
+    residual[(size_t)t * ldr + n] += col_scale ? total * col_scale[n] : total;
   }
 }
 
@@ -322,7 +327,7 @@ int launch_grouped(const GroupedArgs& p, int row_tiles, cudaStream_t stream) {
 }  // namespace
 
 // The general form; see GroupedArgs.  out_f32: C is float32 (else bfloat16); gated 1: W_g has 2N rows
-// and C = act(gate, up) in bfloat16; gated 2: W_g has N rows and C = gelu(A W_g^T) (erf form).  max_rows: an upper bound of the rows over all groups (the
+// and C = act(gate, up) in bfloat16; gated 2 / 3: W_g has N rows and C = gelu(A W_g^T) (erf form) / relu(A W_g^T)^2.  max_rows: an upper bound of the rows over all groups (the
 // grid is sized by it when the counts live on the device).
 GB_EXPORT int gb_grouped_gemm(const void* a, long long lda, long long a_gstride, const int* a_rows, int a_div,
                               const void* w, long long w_gstride, void* c, long long ldc, long long c_gstride,
@@ -332,9 +337,9 @@ GB_EXPORT int gb_grouped_gemm(const void* a, long long lda, long long a_gstride,
   if (groups <= 0 || N <= 0 || max_rows <= 0) return 0;
   if (K <= 0 || K % 8 || lda % 8 || a_gstride % 8 || w_gstride % 8 || ((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return GB_ERR_SIZE;
   if (gated == 1 && out_f32) return GB_ERR_DTYPE;
-  if (gated < 0 || gated > 2) return GB_ERR_ARG;
+  if (gated < 0 || gated > 3) return GB_ERR_ARG;
   GroupedArgs p{(const bf16*)a, lda, a_gstride, a_rows, a_div > 0 ? a_div : 1, (const bf16*)w, w_gstride, c, ldc, c_gstride,
-                scale, scale_rows, s_rstride, s_gstride, offsets, groups, rows, N, K, limit, alpha, shift, gated == 2 ? 1 : 0};
+                scale, scale_rows, s_rstride, s_gstride, offsets, groups, rows, N, K, limit, alpha, shift, gated >= 2 ? gated - 1 : 0};
   const int row_tiles = offsets ? (max_rows + BM - 1) / BM + groups : groups * ((rows + BM - 1) / BM);
   if (gated == 1) return launch_grouped<MODE_GATED, bf16>(p, row_tiles, stream);
   if (out_f32) return launch_grouped<MODE_PLAIN, float>(p, row_tiles, stream);
@@ -368,9 +373,9 @@ GB_EXPORT int gb_moe_permute(const void* h, long long ldh, const int* row_entry,
 }
 
 GB_EXPORT int gb_moe_combine(const float* rows, const int* place, float* residual, long long ldr, int ntok, int width, int top,
-                             cudaStream_t stream) {
+                             const float* col_scale, cudaStream_t stream) {
   if (ntok <= 0) return 0;
-  gb_launch(moe_combine_kernel, dim3(ntok), dim3(256), 0, stream, rows, place, residual, ldr, width, top);
+  gb_launch(moe_combine_kernel, dim3(ntok), dim3(256), 0, stream, rows, place, residual, ldr, width, top, col_scale);
   return gb_launch_status();
 }
 

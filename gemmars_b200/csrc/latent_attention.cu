@@ -19,8 +19,8 @@
 // its position and the cache alone, so prompts, single tokens and any batch give the same bits.
 #include "common.cuh"
 
-// Rotation of interleaved pairs: dims (2i, 2i+1), i < rot/2, angle = float(pos) * inv_freq[i]:
-// (u, v) -> (u cos - v sin, v cos + u sin), all in float32.
+// Rotation of a pair (u, v) -> (u cos - v sin, v cos + u sin), angle = float(pos) * inv_freq[i], all in
+// float32.  Pair i < rot/2 is dims (2i, 2i+1), or with the half layout (i, i + rot/2).
 __device__ __forceinline__ void rotate_pair(float u, float v, float angle, float& ou, float& ov) {
   float s, c;
   sincosf(angle, &s, &c);
@@ -37,7 +37,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
     T* __restrict__ q_lat, long long ldql, float* __restrict__ gate, T* __restrict__ cache,
     const int* __restrict__ page_table, int table_width, int page_size, const int* __restrict__ tok_pos,
     const int* __restrict__ tok_seq, const int* __restrict__ seq_slot, int H, int dim, int rd, int rank,
-    T* __restrict__ dense, long long ldd) {
+    T* __restrict__ dense, long long ldd, int half_layout) {
   __shared__ float scratch[34];
   pdl_release_next();
   pdl_wait_prior();
@@ -65,8 +65,9 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
     for (int i = tid; i < rank; i += blockDim.x) row[i] = from_f32<T>(kv[i] * rstd * norm_w[i]);
     // the shared rotated key part: pairs below `rot` turn, the rest passes
     for (int i = tid; i < rd / 2 + (rd & 1); i += blockDim.x) {
-      const int a = 2 * i, b = 2 * i + 1;
-      if (b < rot) {
+      const bool turns = 2 * i < rot;
+      const int a = turns && half_layout ? i : 2 * i, b = turns && half_layout ? i + rot / 2 : 2 * i + 1;
+      if (turns) {
         float u, v;
         rotate_pair(kv[rank + a], kv[rank + b], fpos * inv_freq[i], u, v);
         row[rank + a] = from_f32<T>(u);
@@ -87,10 +88,11 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
   const int halves = rd / 2 + (rd & 1);
   for (int e = tid; e < H * halves; e += blockDim.x) {
     const int h = e / halves, i = e % halves;
-    const int a = 2 * i, b = 2 * i + 1;
+    const bool turns = 2 * i < rot;
+    const int a = turns && half_layout ? i : 2 * i, b = turns && half_layout ? i + rot / 2 : 2 * i + 1;
     const float* src = q + h * qd + dim;
     T* dst = q_lat + (size_t)t * ldql + (size_t)h * (rank + rd) + rank;
-    if (b < rot) {
+    if (turns) {
       float u, v;
       rotate_pair(src[a], src[b], fpos * inv_freq[i], u, v);
       dst[a] = from_f32<T>(u * q_scale);
@@ -109,14 +111,14 @@ GB_EXPORT int gb_latent_prepare(const float* q_in, long long ldq, const float* k
                                 float q_scale, void* q_nope, long long ldqn, void* q_lat, long long ldql, float* gate,
                                 void* cache, int dtype, const int* page_table, int table_width, int page_size,
                                 const int* tok_pos, const int* tok_seq, const int* seq_slot, int ntok, int H, int dim,
-                                int rd, int rank, void* dense, long long ldd, cudaStream_t stream) {
+                                int rd, int rank, void* dense, long long ldd, int half_layout, cudaStream_t stream) {
   if (ntok <= 0) return 0;
   if (H <= 0 || dim < 0 || rd < 0 || rank <= 0 || rot < 0 || rot > rd || (rot & 1)) return GB_ERR_SIZE;
   if (rot > 0 && inv_freq == nullptr) return GB_ERR_ARG;
 #define LAUNCH(T)                                                                                                     \
   gb_launch(latent_prepare_kernel<T>, dim3(ntok), dim3(256), 0, stream, q_in, ldq, kv_in, ldkv, g_in, ldg, norm_w, eps, \
             inv_freq, rot, q_scale, (T*)q_nope, ldqn, (T*)q_lat, ldql, gate, (T*)cache, page_table, table_width,       \
-            page_size, tok_pos, tok_seq, seq_slot, H, dim, rd, rank, (T*)dense, ldd)
+            page_size, tok_pos, tok_seq, seq_slot, H, dim, rd, rank, (T*)dense, ldd, half_layout)
   if (dtype == GB_F32) LAUNCH(float);
   else if (dtype == GB_BF16) LAUNCH(bf16);
   else return GB_ERR_DTYPE;

@@ -6,9 +6,11 @@
 //              y = g * sigmoid(alpha g) * (u + shift);  out = down y
 //   residual[t] += sum over chosen of weight * expert_e(h[t])  +  sigmoid(sg . h[t]) * shared(h[t])
 //
-// Two more forms for designs that ask for them: `all_softmax` (the weights are the chosen experts'
-// shares of the softmax over ALL experts, not renormalized), and experts without a gate
-// (gb_moe_up: y = gelu(up h) with the exact, erf form; out = down y; the first matrices are [E, ff, width]).
+// Three more forms for designs that ask for them: ROUTE_SOFTMAX_ALL (the weights are the chosen experts'
+// shares of the softmax over ALL experts, not renormalized); ROUTE_SIGMOID (scores s = sigmoid(router . h);
+// chosen by s + bias, weighted by s / (sum of the chosen s + 1e-20) * scale, the bias left out); and
+// experts without a gate (gb_moe_up: y = act(up h), act the exact, erf GELU or the square of relu; out =
+// down y; the first matrices are [E, ff, width]).  `col_scale` [width] multiplies what is added into the residual.
 //
 // The router's logits are a product like any other (the part computes them in float32); this unit
 // picks the experts from them and runs the experts token-major: a block owns one (token, chosen
@@ -70,12 +72,13 @@ template <typename T> __device__ __forceinline__ bool rows_vectorize(const T* ba
 }
 
 // ---- router: the logits come from a product (float32 [ntok, ldz]); a warp per token adds the
-// bias, picks the `top` largest (the lower index wins a tie) and takes the softmax over those
-// alone.  Column E of z, when there is one, is the shared expert's gate logit.
+// bias, picks the `top` largest (the lower index wins a tie) and weighs them as `mode` says (the
+// softmax over those alone by default).  Column E of z, when there is one, is the shared expert's gate logit.
+enum { ROUTE_SOFTMAX_TOP = 0, ROUTE_SOFTMAX_ALL = 1, ROUTE_SIGMOID = 2 };
 __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__ zin, long long ldz,
                                                        const float* __restrict__ bias, int* __restrict__ idx,
                                                        float* __restrict__ wts, float* __restrict__ sg, int ntok, int E,
-                                                       int top, int has_gate, int all_softmax) {
+                                                       int top, int has_gate, int mode, float scale) {
   extern __shared__ float smem[];
   pdl_release_next();
   pdl_wait_prior();
@@ -83,10 +86,14 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__
   const int t = blockIdx.x * 4 + warp;
   if (t >= ntok) return;
   float* z = smem + (size_t)warp * E;
-  for (int e = lane; e < E; e += 32) z[e] = zin[(size_t)t * ldz + e] + (bias ? bias[e] : 0.f);
+  for (int e = lane; e < E; e += 32) {
+    const float v = zin[(size_t)t * ldz + e];
+    z[e] = (mode == ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-v)) : v) + (bias ? bias[e] : 0.f);
+  }
   if (has_gate && lane == 0) sg[t] = 1.0f / (1.0f + expf(-zin[(size_t)t * ldz + E]));
   __syncwarp();
   float mine = 0.f, first = 0.f;   // lane k keeps the k-th chosen logit
+  int mine_at = 0;                 // and whose it is
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int at = 0x7fffffff;
@@ -101,21 +108,27 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__
       if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
     }
     if (k == 0) first = best;
-    if (lane == k) mine = best;
+    if (lane == k) { mine = best; mine_at = at < E ? at : 0; }
     if (lane == 0) {
       idx[(size_t)t * top + k] = at < E ? at : 0;
       if (at < E) z[at] = -INFINITY;
     }
     __syncwarp();
   }
+  if (mode == ROUTE_SIGMOID) {
+    const float s = lane < top ? 1.0f / (1.0f + expf(-zin[(size_t)t * ldz + mine_at])) : 0.f;
+    const float total = warp_sum(s) + 1e-20f;
+    if (lane < top) wts[(size_t)t * top + lane] = s / total * scale;
+    return;
+  }
   const float e = lane < top ? expf(mine - first) : 0.f;
   float sum = warp_sum(e);
-  if (all_softmax) {               // the experts not chosen join the denominator (the chosen ones' places hold -inf: nothing)
+  if (mode == ROUTE_SOFTMAX_ALL) {               // the experts not chosen join the denominator (the chosen ones' places hold -inf: nothing)
     float rest = 0.f;
     for (int i = lane; i < E; i += 32) rest += expf(z[i] - first);
     sum += warp_sum(rest);
   }
-  if (lane < top) wts[(size_t)t * top + lane] = e / sum;
+  if (lane < top) wts[(size_t)t * top + lane] = e / sum * scale;
 }
 
 // ---- gate and up of one (token, slot): FEATS features a block, a warp per feature in turn
@@ -155,12 +168,16 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(const T* __restrict__ 
   }
 }
 
-// ---- the same for experts without a gate: y = gelu(up h) (erf form), two features a warp at a time
-__device__ __forceinline__ float gelu_erf_f(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f)); }
+// ---- the same for experts without a gate: y = act(up h), two features a warp at a time
+enum { ACT_GELU = 1, ACT_RELU2 = 2 };     // the exact (erf) GELU; the square of relu
+__device__ __forceinline__ float plain_act(float x, int act) {
+  if (act == ACT_RELU2) return fmaxf(x, 0.f) * fmaxf(x, 0.f);
+  return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f));
+}
 
 template <typename T>
 __global__ void __launch_bounds__(256) moe_up_kernel(const T* __restrict__ h, long long ldh, const int* __restrict__ idx,
-                                                     const T* __restrict__ w_up, T* __restrict__ y, int width, int ff, int top) {
+                                                     const T* __restrict__ w_up, T* __restrict__ y, int width, int ff, int top, int act) {
   extern __shared__ float xs[];   // [width]
   pdl_release_next();
   pdl_wait_prior();
@@ -179,8 +196,8 @@ __global__ void __launch_bounds__(256) moe_up_kernel(const T* __restrict__ h, lo
     a = warp_sum(a);
     b = warp_sum(b);
     if (lane == 0) {
-      y[((size_t)t * top + s) * ff + f] = from_f32<T>(gelu_erf_f(a));
-      if (two) y[((size_t)t * top + s) * ff + f + 1] = from_f32<T>(gelu_erf_f(b));
+      y[((size_t)t * top + s) * ff + f] = from_f32<T>(plain_act(a, act));
+      if (two) y[((size_t)t * top + s) * ff + f + 1] = from_f32<T>(plain_act(b, act));
     }
   }
 }
@@ -220,29 +237,31 @@ __global__ void __launch_bounds__(256) moe_down_kernel(const T* __restrict__ y, 
 }
 
 __global__ void __launch_bounds__(256) moe_sum_kernel(const float* __restrict__ rows, float* __restrict__ residual,
-                                                      long long ldr, int width, int slots) {
+                                                      long long ldr, int width, int slots,
+                                                      const float* __restrict__ col_scale) {
   pdl_release_next();
   pdl_wait_prior();
   const int t = blockIdx.x;
   for (int n = blockIdx.y * 256 + threadIdx.x; n < width; n += gridDim.y * 256) {
     float total = 0.f;
     for (int s = 0; s < slots; ++s) total += rows[((size_t)t * slots + s) * width + n];
-    residual[(size_t)t * ldr + n] += total;
+    residual[(size_t)t * ldr + n] += col_scale ? total * col_scale[n] : total;
   }
 }
 
 GB_EXPORT int gb_moe_topk_mode(const float* z, long long ldz, const float* bias, int* idx, float* wts, float* sg, int ntok,
-                               int E, int top, int has_gate, int all_softmax, cudaStream_t stream) {
+                               int E, int top, int has_gate, int mode, float scale, cudaStream_t stream) {
   if (ntok <= 0) return 0;
+  if (mode < ROUTE_SOFTMAX_TOP || mode > ROUTE_SIGMOID) return GB_ERR_ARG;
   if (E <= 0 || top <= 0 || top > 32 || top > E || E > 2048) return GB_ERR_SIZE;
   gb_launch(moe_topk_kernel, dim3((ntok + 3) / 4), dim3(128), (size_t)4 * E * sizeof(float), stream, z, ldz, bias, idx, wts, sg,
-            ntok, E, top, has_gate, all_softmax);
+            ntok, E, top, has_gate, mode, scale);
   return gb_launch_status();
 }
 
 GB_EXPORT int gb_moe_topk(const float* z, long long ldz, const float* bias, int* idx, float* wts, float* sg, int ntok,
                           int E, int top, int has_gate, cudaStream_t stream) {
-  return gb_moe_topk_mode(z, ldz, bias, idx, wts, sg, ntok, E, top, has_gate, 0, stream);
+  return gb_moe_topk_mode(z, ldz, bias, idx, wts, sg, ntok, E, top, has_gate, ROUTE_SOFTMAX_TOP, 1.0f, stream);
 }
 
 // w_gu: [E, 2 ff, width] (an expert's gate rows, then its up rows); ws_gu: [2 ffs, width] or null;
@@ -267,20 +286,21 @@ GB_EXPORT int gb_moe_gate_up(const void* h, long long ldh, int dtype, const int*
   return gb_launch_status();
 }
 
-// Experts without a gate: w_up [E, ff, width]; y: [ntok, top, ff] = gelu(up h) of every chosen expert.
+// Experts without a gate: w_up [E, ff, width]; y: [ntok, top, ff] = act(up h) of every chosen expert.
 GB_EXPORT int gb_moe_up(const void* h, long long ldh, int dtype, const int* idx, const void* w_up, void* y, int ntok, int width,
-                        int ff, int top, cudaStream_t stream) {
+                        int ff, int top, int act, cudaStream_t stream) {
   if (ntok <= 0) return 0;
+  if (act != ACT_GELU && act != ACT_RELU2) return GB_ERR_ARG;
   if (width <= 0 || ff <= 0 || top <= 0) return GB_ERR_SIZE;
   const size_t smem = (size_t)width * sizeof(float);
   if (smem > 48 * 1024) return GB_ERR_SIZE;
   dim3 grid(ntok * top, (ff + FEATS - 1) / FEATS);
   if (dtype == GB_F32)
     gb_launch(moe_up_kernel<float>, grid, dim3(256), smem, stream, (const float*)h, ldh, idx, (const float*)w_up, (float*)y,
-              width, ff, top);
+              width, ff, top, act);
   else if (dtype == GB_BF16)
     gb_launch(moe_up_kernel<bf16>, grid, dim3(256), smem, stream, (const bf16*)h, ldh, idx, (const bf16*)w_up, (bf16*)y, width,
-              ff, top);
+              ff, top, act);
   else
     return GB_ERR_DTYPE;
   return gb_launch_status();
@@ -290,7 +310,7 @@ GB_EXPORT int gb_moe_up(const void* h, long long ldh, int dtype, const int* idx,
 // residual: float32 [ntok, width] rows ldr apart.
 GB_EXPORT int gb_moe_down(const void* y, int dtype, const int* idx, const float* wts, const float* sg, const void* w_d,
                           const void* ws_d, float* rows, float* residual, long long ldr, int ntok, int width, int ff, int ffs,
-                          int top, cudaStream_t stream) {
+                          int top, const float* col_scale, cudaStream_t stream) {
   if (ntok <= 0) return 0;
   const int slots = top + (ws_d ? 1 : 0), ffmax = ff > ffs ? ff : ffs;
   if (width <= 0 || ffmax <= 0 || slots <= 0) return GB_ERR_SIZE;
@@ -306,6 +326,6 @@ GB_EXPORT int gb_moe_down(const void* y, int dtype, const int* idx, const float*
   else
     return GB_ERR_DTYPE;
   gb_launch(moe_sum_kernel, dim3(ntok, (width + 1023) / 1024), dim3(256), 0, stream, (const float*)rows, residual, ldr, width,
-            slots);
+            slots, col_scale);
   return gb_launch_status();
 }

@@ -1,6 +1,7 @@
 // Kernels of the mixers that carry a fixed-size state from token to token: the short causal
 // filter over time, the gated delta rule, the selective state-space recurrence with a scalar
-// decay per head, and the gated RMS norm over groups of channels that follows them.
+// decay per head, linear attention with a decay per key channel, matrix memory with exponential gates,
+// and the gated RMS norm over groups of channels that follows them.
 //
 // A step's tokens are packed; sequence b owns rows cu[b] .. cu[b+1]-1 and the state row
 // seq_slot[b].  Every kernel walks a sequence's rows in order on the device, so a whole prompt, a
@@ -913,4 +914,162 @@ GB_EXPORT int gb_wkv_scan(const float* r, const float* k, const float* w, long l
                           const float* bonus, float* state, const int* cu, const int* seq_slot, float* y, int nseq, int H, int D,
                           int V, cudaStream_t stream) {
   return gb_wkv_scan_scaled(r, k, w, ld, ld, v, ldv, bonus, state, cu, seq_slot, y, nseq, H, D, V, 1.0f, stream);
+}
+
+// ------------------------------------------------------------------ matrix memory with exponential gates
+// The state of a head is a matrix S [dim, vdim], a vector n [dim] and a running maximum m; blocks,
+// columns, lanes and the order of S in memory as for the delta rule (dim <= 32 P).  Per token, with
+// i = cap tanh(il / cap) and f = logsigmoid(cap tanh(fl / cap)) of the gates' logits (cap 0: no cap):
+//   m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  n <- the same with k alone;
+//   y = S^T (qscale q) / (max(|n . (qscale q)|, exp(-m')) + 1e-6)
+// Tokens come in groups of GR by asynchronous copies, a group ahead.  For a group at once, before the
+// walk over its tokens: the gates (a token a thread), the running maximum (a sum and a maximum a
+// token, every lane of a warp the same, its exponentials a token a lane), and n with its products
+// n . q: thread d keeps n[d], so a token costs it two multiplications and a share of a sum that only
+// has to be there when the walk begins.  A block of 32 columns keeps an n and an m of its own
+// (aux [slots, H, blocks, 32 P + 4]: n, then m), since blocks of one head may run one after the other.
+template <int P, int GR>
+__global__ void __launch_bounds__(32 * P) matrix_memory_kernel(const float* __restrict__ q, const float* __restrict__ k,
+                                                              const float* __restrict__ v, const float* __restrict__ in_logit,
+                                                              const float* __restrict__ forget_logit, long long ld,
+                                                              float* __restrict__ state, float* __restrict__ aux,
+                                                              const int* __restrict__ cu, const int* __restrict__ seq_slot,
+                                                              float* __restrict__ y, int H, int D, int V, float cap, float qscale) {
+  constexpr int DP = P * SLICE;
+  __shared__ __align__(16) float kq[2][GR][2][padded_size(P)];   // [buffer][token][k | q][dims, padded]
+  __shared__ float vs[2][GR][32], gates[2][GR][2];
+  __shared__ float logs[GR][2], pre[GR][3];                      // i and f; then: what S keeps, what is written, exp(-m)
+  __shared__ float nq[GR][P];                                    // the warps' shares of n . q
+  pdl_wait_prior();
+  const int b = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
+  const int col = blockIdx.z * 32 + tid / P, part = tid % P, lane = tid & 31, warp = tid >> 5;
+  const bool live = col < V;
+  const int t0 = cu[b], t1 = cu[b + 1];
+  float4* Sg = (float4*)(state + ((size_t)seq_slot[b] * H + head) * 8 * V * P * 4);
+  float* ax = aux + (((size_t)seq_slot[b] * H + head) * gridDim.z + blockIdx.z) * (DP + 4);
+  float S[SLICE];
+#pragma unroll
+  for (int r = 0; r < SLICE / 4; ++r) {
+    const float4 s4 = live ? Sg[((size_t)r * V + col) * P + part] : make_float4(0.f, 0.f, 0.f, 0.f);
+    S[4 * r] = s4.x; S[4 * r + 1] = s4.y; S[4 * r + 2] = s4.z; S[4 * r + 3] = s4.w;
+  }
+  float nd = ax[tid], m = ax[DP];
+  if (tid >= D)      // the dims beyond the head's are zeros, written once
+    for (int j = 0; j < 2 * GR; ++j) kq[j / GR][j % GR][0][padded(tid)] = kq[j / GR][j % GR][1][padded(tid)] = 0.f;
+  auto bring = [&](int first, int buf) {
+    for (int j = 0; j < GR && first + j < t1; ++j) {
+      const size_t t = first + j;
+      if (tid < D) {
+        copy_async4(&kq[buf][j][0][padded(tid)], k + t * ld + head * D + tid);
+        copy_async4(&kq[buf][j][1][padded(tid)], q + t * ld + head * D + tid);
+      }
+      if (live && part == 0) copy_async4(&vs[buf][j][tid / P], v + t * ld + head * V + col);
+      if (tid == 0) copy_async4(&gates[buf][j][0], in_logit + t * ld + head);
+      if (tid == 1) copy_async4(&gates[buf][j][1], forget_logit + t * ld + head);
+    }
+    copy_async_commit();
+  };
+  bring(t0, 0);
+  for (int first = t0; first < t1; first += GR) {
+    const int buf = ((first - t0) / GR) & 1;
+    if (first + GR < t1) {
+      bring(first + GR, buf ^ 1);
+      copy_async_wait<1>();
+    } else {
+      copy_async_wait<0>();
+    }
+    __syncthreads();
+    const int n = min(GR, t1 - first);
+    if (tid < 2 * n) {                        // a gate a thread: 2 GR <= 32, so one warp has them all
+      const int j = tid >> 1;
+      float z = gates[buf][j][tid & 1];
+      if (cap > 0.f) z = cap * tanhf(z / cap);
+      logs[j][tid & 1] = (tid & 1) ? -softplus_f(-z) : z;
+    }
+    __syncthreads();
+    {                                         // every warp takes the maxima for itself; warp 0 leaves the factors
+      float before = m, mine_before = 0.f, mine = 0.f;
+      for (int j = 0; j < n; ++j) {
+        const float now = fmaxf(logs[j][1] + before, logs[j][0]);
+        if (lane == j) { mine_before = before; mine = now; }
+        before = now;
+      }
+      m = before;
+      float keep = 0.f, write = 0.f;
+      if (lane < n) {
+        keep = expf(logs[lane][1] + mine_before - mine);
+        write = expf(logs[lane][0] - mine);
+        if (warp == 0) {
+          pre[lane][0] = keep;
+          pre[lane][1] = write;
+          pre[lane][2] = expf(-mine);
+        }
+      }
+      for (int j = 0; j < n; ++j) {
+        const float kp = __shfl_sync(0xffffffffu, keep, j), wr = __shfl_sync(0xffffffffu, write, j);
+        nd = fmaf(wr, kq[buf][j][0][padded(tid)], kp * nd);
+        const float s = warp_sum(nd * kq[buf][j][1][padded(tid)]);
+        if (lane == 0) nq[j][warp] = s;
+      }
+    }
+    __syncthreads();
+    for (int j = 0; j < n; ++j) {
+      const float4* ks = (const float4*)(kq[buf][j][0] + part * (SLICE + 4));
+      const float4* qs = (const float4*)(kq[buf][j][1] + part * (SLICE + 4));
+      const float keep = pre[j][0], wv = pre[j][1] * (live ? vs[buf][j][tid / P] : 0.f);
+      float acc = 0.f, acc2 = 0.f;
+#pragma unroll
+      for (int r = 0; r < SLICE / 4; ++r) {
+        const float4 kv = ks[r], qv = qs[r];
+        S[4 * r] = fmaf(kv.x, wv, keep * S[4 * r]);         acc = fmaf(S[4 * r], qv.x, acc);
+        S[4 * r + 1] = fmaf(kv.y, wv, keep * S[4 * r + 1]); acc2 = fmaf(S[4 * r + 1], qv.y, acc2);
+        S[4 * r + 2] = fmaf(kv.z, wv, keep * S[4 * r + 2]); acc = fmaf(S[4 * r + 2], qv.z, acc);
+        S[4 * r + 3] = fmaf(kv.w, wv, keep * S[4 * r + 3]); acc2 = fmaf(S[4 * r + 3], qv.w, acc2);
+      }
+      acc = lanes_sum<P>(acc + acc2);
+      if (live && part == 0) {
+        float dot = nq[j][0];
+#pragma unroll
+        for (int w = 1; w < P; ++w) dot += nq[j][w];
+        y[(size_t)(first + j) * H * V + head * V + col] = acc * qscale / (fmaxf(fabsf(dot * qscale), pre[j][2]) + 1e-6f);
+      }
+    }
+    __syncthreads();   // the group after next is brought into this buffer; pre and nq are written again
+  }
+  // only now may the kernel after this one start: its waiting blocks would take the room of this
+  // kernel's few warps, which are a chain from token to token
+  pdl_release_next();
+  ax[tid] = nd;
+  if (tid == 0) ax[DP] = m;
+  if (live) {
+#pragma unroll
+    for (int r = 0; r < SLICE / 4; ++r)
+      Sg[((size_t)r * V + col) * P + part] = make_float4(S[4 * r], S[4 * r + 1], S[4 * r + 2], S[4 * r + 3]);
+  }
+}
+
+// Floats of one head's n and m (what a caller allocates per slot and head): one set per 32 columns.
+GB_EXPORT int gb_matrix_memory_aux_floats(int dims, int V) { return (V + 31) / 32 * (lanes_for(dims) * SLICE + 4); }
+
+// q, k: rows of ld floats, head h at h * D; v: head h at h * V; in_logit, forget_logit: [ntok, H] in rows of ld;
+// state: [slots, H, gb_state_floats(D, V)], aux: [slots, H, gb_matrix_memory_aux_floats(D, V)] float32, zeros
+// for a new sequence; y: [ntok, H * V].  cap: the gates' cap (0: none).
+GB_EXPORT int gb_matrix_memory(const float* q, const float* k, const float* v, const float* in_logit, const float* forget_logit,
+                               long long ld, float* state, float* aux, const int* cu, const int* seq_slot, float* y, int nseq,
+                               int H, int D, int V, float cap, float qscale, cudaStream_t stream) {
+  if (nseq <= 0) return 0;
+  if (H <= 0 || V <= 0 || D <= 0 || D > 8 * SLICE || ((uintptr_t)state & 15)) return GB_ERR_SIZE;
+  if (cap < 0.f) return GB_ERR_ARG;
+  dim3 grid(nseq, H, (V + 31) / 32);
+#define GB_MEMORY(P, GR)                                                                                                \
+  launch_scan(matrix_memory_kernel<P, GR>, grid, 32 * P, stream, q, k, v, in_logit, forget_logit, ld, state, aux, cu, seq_slot, y, \
+              H, D, V, cap, qscale)
+  switch (lanes_for(D)) {
+    case 1: GB_MEMORY(1, 8); break;
+    case 2: GB_MEMORY(2, 8); break;
+    case 4: GB_MEMORY(4, 8); break;
+    default: GB_MEMORY(8, 8);
+  }
+#undef GB_MEMORY
+  return gb_launch_status();
 }

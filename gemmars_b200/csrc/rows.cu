@@ -3,7 +3,10 @@
 //  * an RMSNorm applied to a sublayer's OUTPUT and added into the stream (norms on both sides of
 //    a sublayer): x[t] += y[t] * (mean(y[t]^2) + eps)^-1/2 * w;
 //  * the gated activation act(g) * u for a choice of act;
-//  * a scale on float32 rows (logits).
+//  * a scale on float32 rows, and a cap cap * tanh(y / cap) (logits);
+//  * a gathered table row that is normed before it becomes the stream (an embedding with a norm);
+//  * one row added to every row of the stream, with the norm that reads the stream next;
+//  * an RMSNorm of a slice of columns (the latent inside a mixer).
 // Statistics, sums and the activation's arithmetic are float32.
 #include "common.cuh"
 
@@ -159,5 +162,145 @@ GB_EXPORT int gb_scale_f32(float* y, long long total, float s, cudaStream_t stre
   if (total <= 0) return 0;
   const int blocks = (int)((total + 255) / 256 < 2048 ? (total + 255) / 256 : 2048);
   gb_launch(scale_kernel, blocks, 256, 0, stream, y, total, s);
+  return gb_launch_status();
+}
+
+// y = cap * tanh(y / cap)
+__global__ void cap_kernel(float* __restrict__ y, long long total, float cap) {
+  pdl_release_next();
+  pdl_wait_prior();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x)
+    y[i] = cap * tanhf(y[i] / cap);
+}
+
+GB_EXPORT int gb_cap_f32(float* y, long long total, float cap, cudaStream_t stream) {
+  if (total <= 0) return 0;
+  if (!(cap > 0.f)) return GB_ERR_ARG;
+  const int blocks = (int)((total + 255) / 256 < 2048 ? (total + 255) / 256 : 2048);
+  gb_launch(cap_kernel, blocks, 256, 0, stream, y, total, cap);
+  return gb_launch_status();
+}
+
+// One block a row: in(i) gives the row's element i, out(i, normed) takes it.  The row is kept in
+// registers between the passes where it fits, else read again; the order of the additions depends on
+// n and the block size alone.
+template <typename In, typename Out>
+__device__ __forceinline__ void norm_row(int n, float eps, float* scratch, In in, Out out) {
+  constexpr int KEEP = 8;
+  float held[KEEP], ss = 0.f;
+  const bool keep = n <= KEEP * (int)blockDim.x;
+  if (keep) {
+#pragma unroll
+    for (int u = 0; u < KEEP; ++u) {
+      const int i = threadIdx.x + u * blockDim.x;
+      held[u] = i < n ? in(i) : 0.f;
+      ss = fmaf(held[u], held[u], ss);
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      const float v = in(i);
+      ss = fmaf(v, v, ss);
+    }
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+  if (keep) {
+#pragma unroll
+    for (int u = 0; u < KEEP; ++u) {
+      const int i = threadIdx.x + u * blockDim.x;
+      if (i < n) out(i, held[u] * inv);
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) out(i, in(i) * inv);
+  }
+}
+static inline int row_threads(int n) { return n >= 2048 ? 512 : (n >= 512 ? 256 : 128); }
+
+// x[t, :] = rmsnorm(table[tokens[t], :] * scale) * w
+template <typename W>
+__global__ void __launch_bounds__(512) embed_norm_kernel(const W* __restrict__ table, const int* __restrict__ tokens,
+                                                         const float* __restrict__ w, float* __restrict__ x, int hidden, int rows,
+                                                         float scale, float eps) {
+  __shared__ float scratch[33];
+  pdl_release_next();
+  pdl_wait_prior();
+  int id = tokens[blockIdx.x];
+  id = id < 0 ? 0 : (id >= rows ? rows - 1 : id);
+  const W* row = table + (size_t)id * hidden;
+  float* out = x + (size_t)blockIdx.x * hidden;
+  norm_row(hidden, eps, scratch, [&](int i) { return to_f32(row[i]) * scale; }, [&](int i, float v) { out[i] = v * w[i]; });
+}
+
+GB_EXPORT int gb_embed_norm(const void* table, int table_dtype, const int* tokens, const float* w, float* x, int ntok, int hidden,
+                            int rows, float scale, float eps, cudaStream_t stream) {
+  if (ntok <= 0) return 0;
+  if (hidden <= 0 || rows <= 0) return GB_ERR_SIZE;
+  const int threads = row_threads(hidden);
+  if (table_dtype == GB_F32)
+    gb_launch(embed_norm_kernel<float>, ntok, threads, 0, stream, (const float*)table, tokens, w, x, hidden, rows, scale, eps);
+  else if (table_dtype == GB_BF16)
+    gb_launch(embed_norm_kernel<bf16>, ntok, threads, 0, stream, (const bf16*)table, tokens, w, x, hidden, rows, scale, eps);
+  else
+    return GB_ERR_DTYPE;
+  return gb_launch_status();
+}
+
+// x[t, :] += v for every row, and, when a weight is given, h[t, :] = rmsnorm(x[t, :]) * w of the new rows
+template <typename O>
+__global__ void __launch_bounds__(512) add_row_norm_kernel(const float* __restrict__ v, float* __restrict__ x, int n,
+                                                           const float* __restrict__ w, O* __restrict__ h, float eps) {
+  __shared__ float scratch[33];
+  pdl_release_next();
+  pdl_wait_prior();
+  float* row = x + (size_t)blockIdx.x * n;
+  if (!w) {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) row[i] += v[i];
+    return;
+  }
+  O* hrow = h + (size_t)blockIdx.x * n;
+  // a thread reads, in both passes of a long row, only elements that it wrote or that nobody has written yet
+  norm_row(n, eps, scratch, [&](int i) { return row[i] + v[i]; },
+           [&](int i, float normed) {
+             hrow[i] = from_f32<O>(normed * w[i]);
+             row[i] += v[i];
+           });
+}
+
+GB_EXPORT int gb_add_row_norm(const float* v, float* x, int rows, int n, const float* w, void* h, int h_dtype, float eps,
+                              cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (n <= 0) return GB_ERR_SIZE;
+  const int threads = row_threads(n);
+  if (w && h_dtype == GB_BF16)
+    gb_launch(add_row_norm_kernel<bf16>, rows, threads, 0, stream, v, x, n, w, (bf16*)h, eps);
+  else if (!w || h_dtype == GB_F32)
+    gb_launch(add_row_norm_kernel<float>, rows, threads, 0, stream, v, x, n, w, (float*)h, eps);
+  else
+    return GB_ERR_DTYPE;
+  return gb_launch_status();
+}
+
+// out[t, :] = rmsnorm(x[t, :n]) * w for rows of x that are ldx floats apart
+template <typename O>
+__global__ void __launch_bounds__(512) norm_cols_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w,
+                                                        O* __restrict__ out, int n, float eps) {
+  __shared__ float scratch[33];
+  pdl_release_next();
+  pdl_wait_prior();
+  const float* row = x + (size_t)blockIdx.x * ldx;
+  O* o = out + (size_t)blockIdx.x * n;
+  norm_row(n, eps, scratch, [&](int i) { return row[i]; }, [&](int i, float v) { o[i] = from_f32<O>(v * w[i]); });
+}
+
+GB_EXPORT int gb_norm_cols(const float* x, long long ldx, const float* w, void* out, int out_dtype, int rows, int n, float eps,
+                           cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (n <= 0) return GB_ERR_SIZE;
+  const int threads = row_threads(n);
+  if (out_dtype == GB_F32)
+    gb_launch(norm_cols_kernel<float>, rows, threads, 0, stream, x, ldx, w, (float*)out, n, eps);
+  else if (out_dtype == GB_BF16)
+    gb_launch(norm_cols_kernel<bf16>, rows, threads, 0, stream, x, ldx, w, (bf16*)out, n, eps);
+  else
+    return GB_ERR_DTYPE;
   return gb_launch_status();
 }

@@ -28,6 +28,7 @@ class DecoderModel:
         self.act_dtype = compute_dtype(compute)
         self.embedding = build_part("embedding", plan.embedding, compute)
         self.blocks = [build_block(ls, compute) for ls in plan.layers]
+        self.before = [build_part("stream", e.before, compute) if e.before is not None else None for e in plan.schedule]
         self.final_norm = build_part("norm", plan.final_norm, compute)
         self.head = build_part("head", plan.head, compute)
         self.config = None
@@ -40,6 +41,9 @@ class DecoderModel:
         yield self.embedding, self.plan.embedding
         for block in self.blocks:
             for part in block.parts().values():
+                yield part, part.spec
+        for part in self.before:
+            if part is not None:
                 yield part, part.spec
         yield self.final_norm, self.plan.final_norm
         yield self.head, self.plan.head
@@ -139,9 +143,14 @@ class DecoderModel:
             owner = i if e.cache_of is None else e.cache_of
             block = self.blocks[e.layer]
             ctx.extras["entry"] = i
-            if getattr(block, "chains_norms", False):
-                after = self.blocks[schedule[i + 1].layer] if i + 1 < len(schedule) else None
-                next_norm = after.first_norm() if getattr(after, "chains_norms", False) else None
+            chains = getattr(block, "chains_norms", False)
+            if self.before[i] is not None:
+                carry = self.before[i].forward(ctx, x, then_norm=block.first_norm() if chains else None)
+            if chains:
+                # a norm is left for the next run only if nothing changes the stream in between
+                after = self.blocks[schedule[i + 1].layer] if i + 1 < len(schedule) and self.before[i + 1] is None else None
+                takes = getattr(after, "chains_norms", False) and after.takes_unscaled_rows
+                next_norm = after.first_norm() if takes else None
                 carry = block.forward(ctx, x, ctx.cache.views(owner), writes_cache=e.cache_of is None, h_in=carry,
                                       next_norm=next_norm)
             else:
@@ -161,6 +170,7 @@ class DecoderModel:
         for e in self.plan.schedule:
             runs[e.layer] = runs.get(e.layer, 0) + 1
         total = self.embedding.weight_bytes() + self.final_norm.weight_bytes() + self.head.weight_bytes()
+        total += sum(part.weight_bytes() for part in self.before if part is not None)
         for i, block in enumerate(self.blocks):
             total += runs.get(i, 0) * sum(part.weight_bytes() for part in block.parts().values())
         return total

@@ -246,10 +246,22 @@ def silu_mul(gu: torch.Tensor, out: torch.Tensor):
 
 # --------------------------------------------------------------------------- matrix products
 
-def gemm_ref(x, w, out, bias=None, accumulate=False):
+#: activations of a product without a gate: the exact (erf) GELU, the square of relu
+PLAIN_ACTS = {None: 0, "gelu": 1, "relu2": 2}
+
+
+def _check_col_scale(col_scale, n, accumulate=True):
+    if col_scale is not None:
+        _cuda(col_scale)
+        assert col_scale.dtype == torch.float32 and col_scale.is_contiguous() and col_scale.numel() == n and accumulate
+
+
+def gemm_ref(x, w, out, bias=None, accumulate=False, act=None, col_scale=None):
     """out = x @ w.T (+ bias), or out += ... (float32 out) with ``accumulate``; CUDA cores, float32
-    accumulation in ascending order of the inner index."""
+    accumulation in ascending order of the inner index.  ``act`` (one of PLAIN_ACTS) is applied to
+    the result; ``col_scale`` (float32 [N], with ``accumulate``) multiplies what is added."""
     _cuda(x, w, out, bias)
+    _check_col_scale(col_scale, w.shape[0], accumulate)
     assert x.dtype == w.dtype and x.stride(-1) == 1 and out.stride(-1) == 1 and w.is_contiguous()
     m, k = x.shape
     n = w.shape[0]
@@ -258,9 +270,10 @@ def gemm_ref(x, w, out, bias=None, accumulate=False):
         assert bias.dtype == torch.float32 and bias.numel() == n
     f = _fn("gemm_ref", "gb_gemm_ref",
             [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_longlong,
-             c_longlong, c_void_p])
+             c_longlong, c_int, c_void_p, c_void_p])
     _check(f(x.data_ptr(), w.data_ptr(), dtype_code(x.dtype), _ptr(bias), out.data_ptr(), dtype_code(out.dtype),
-             OUT_ACCUMULATE if accumulate else OUT_STORE, m, n, k, x.stride(0), out.stride(0), _stream()), "gemm_ref",
+             OUT_ACCUMULATE if accumulate else OUT_STORE, m, n, k, x.stride(0), out.stride(0), PLAIN_ACTS[act],
+             _ptr(col_scale), _stream()), "gemm_ref",
            "matmul", _nbytes(x, w, bias, out) * 1 + (_nbytes(out) if accumulate else 0))
 
 
@@ -368,13 +381,15 @@ GATED_ACT_DEFINES = {"silu": (), "gelu_tanh": (("GB_GATED_ACT", 1),)}
 
 
 def gemm_tc(x, w, out, bias=None, accumulate=False, bn=None, splits=None, stages=4, swiglu=False, link_in=None,
-            link_out=None, act="silu"):
+            link_out=None, act="silu", plain_act=None, col_scale=None):
     """out = x @ w.T (+ bias) (bfloat16 or float32 out) or out += ... (float32 out), bfloat16
     operands, on the tcgen05 tensor cores.  With ``swiglu``, w stacks a gate matrix over an up
     matrix ([2N, K]) and out[M, N] = silu(x @ gate.T) * (x @ up.T) in bfloat16.
     ``link_in``: an UnscaledRows whose ``rows`` are x: every token's results are scaled by its
     rstd.  ``link_out`` = (norm weight float32 [N], eps): with ``accumulate``, also leaves
-    bfloat16(out * weight) and the sums of squares of out's rows, returned as UnscaledRows."""
+    bfloat16(out * weight) and the sums of squares of out's rows, returned as UnscaledRows.
+    ``plain_act`` (one of PLAIN_ACTS, bfloat16 out): applied to the results before they are rounded.
+    ``col_scale`` (float32 [N], with ``accumulate``): multiplies what is added."""
     if link_in is not None:
         assert x is link_in.rows
     _cuda(x, w, out, bias)
@@ -394,8 +409,9 @@ def gemm_tc(x, w, out, bias=None, accumulate=False, bn=None, splits=None, stages
         raise KernelError(f"gemm_tc: cannot {'add into' if accumulate else 'store'} {out.dtype}")
     if bias is not None:
         assert bias.dtype == torch.float32 and bias.numel() == n
+    _check_col_scale(col_scale, n, accumulate)
     auto_bn, auto_splits = gemm_tc_tiling(m, n, k, gated=swiglu)
-    if link_in is None and link_out is None:
+    if link_in is None and link_out is None and plain_act is None and col_scale is None:
         f = _fn("gemm_tc", "gb_gemm_tc",
                 [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_int,
                  c_int, c_int, c_void_p], GATED_ACT_DEFINES[act] if swiglu else ())
@@ -403,7 +419,7 @@ def gemm_tc(x, w, out, bias=None, accumulate=False, bn=None, splits=None, stages
                  bn or auto_bn, splits or auto_splits, stages, _stream()), "gemm_tc", "matmul",
                _nbytes(x, w, bias, out) + (_nbytes(out) if accumulate else 0))
         return None
-    if m > LINK_MAX_TOKENS:
+    if m > LINK_MAX_TOKENS and (link_in is not None or link_out is not None):
         raise KernelError(f"gemm_tc: a norm can be taken into the product for at most {LINK_MAX_TOKENS} tokens")
     left = None
     if link_out is not None:
@@ -416,7 +432,8 @@ def gemm_tc(x, w, out, bias=None, accumulate=False, bn=None, splits=None, stages
                             torch.empty((-(-n // 128), 64), dtype=torch.float32, device=x.device), eps, n)
     f = _fn("gemm_tc", "gb_gemm_tc_linked",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_int,
-             c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p])
+             c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p,
+             c_void_p], GATED_ACT_DEFINES[act] if swiglu else ())
     _check(f(x.data_ptr(), w.data_ptr(), _ptr(bias), out.data_ptr(), mode, m, n, k, x.stride(0), out.stride(0),
              bn or auto_bn, splits or auto_splits, stages,
              link_in.partial.data_ptr() if link_in is not None else None,
@@ -424,7 +441,7 @@ def gemm_tc(x, w, out, bias=None, accumulate=False, bn=None, splits=None, stages
              link_in.width if link_in is not None else 0,
              link_out[0].data_ptr() if left is not None else None, left.rows.data_ptr() if left is not None else None,
              left.rows.stride(0) if left is not None else 0, left.partial.data_ptr() if left is not None else None,
-             _stream()), "gemm_tc", "matmul",
+             PLAIN_ACTS[plain_act], _ptr(col_scale), _stream()), "gemm_tc", "matmul",
            _nbytes(x, w, bias, out) + (_nbytes(out) if accumulate else 0) + (_nbytes(left.rows) if left is not None else 0))
     return left
 
@@ -434,12 +451,13 @@ PERSISTENT_SPLIT_LAST_ROUND = True
 
 
 def gemm_tc_persistent(x, w, out, bias=None, accumulate=False, swiglu=False, bn=None, ctas=None, split_last=None,
-                       act="silu"):
+                       act="silu", plain_act=None, col_scale=None):
     """The tensor-core product for prompts (more than 64 rows of x): one CTA per SM walks the output
     tiles, and the epilogue of a tile runs while the next tile's MMAs fill the other accumulator
     buffer.  Operands and modes as gemm_tc.  Where the last round of tiles would leave SMs idle, a
     product that adds into ``out`` cuts that round's tiles into parts along the inner dimension,
-    which are added in a fixed order (``split_last=False``: never)."""
+    which are added in a fixed order (``split_last=False``: never).  ``plain_act``, ``col_scale``: as
+    gemm_tc."""
     if split_last is None:
         split_last = PERSISTENT_SPLIT_LAST_ROUND
     _cuda(x, w, out, bias)
@@ -476,9 +494,10 @@ def gemm_tc_persistent(x, w, out, bias=None, accumulate=False, swiglu=False, bn=
             flags = _part_flags[x.device.index] = torch.zeros(max(4 * ctas, 1024), dtype=torch.int32, device=x.device)
     f = _fn("gemm_tc", "gb_gemm_tc_persistent",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_int,
-             c_int, c_void_p, c_void_p], GATED_ACT_DEFINES[act] if swiglu else ())
+             c_int, c_void_p, c_int, c_void_p, c_void_p], GATED_ACT_DEFINES[act] if swiglu else ())
+    _check_col_scale(col_scale, n, accumulate)
     _check(f(x.data_ptr(), w.data_ptr(), _ptr(bias), out.data_ptr(), mode, m, n, k, x.stride(0), out.stride(0), bn,
-             ctas, _ptr(flags), _stream()), "gemm_tc_persistent", "matmul",
+             ctas, _ptr(flags), PLAIN_ACTS[plain_act], _ptr(col_scale), _stream()), "gemm_tc_persistent", "matmul",
            _nbytes(x, w, bias, out) + (_nbytes(out) if accumulate else 0))
 
 
@@ -848,10 +867,10 @@ def attention_prefill_tc_status(head_dim: int = 0, reset: bool = True) -> int:
 # --------------------------------------------------------------------------- latent attention
 
 def latent_prepare(q_in, kv_in, g_in, norm_w, eps, inv_freq, rot, q_scale, q_nope, q_lat, gate, cache, page_table,
-                   page_size, tok_pos, tok_seq, seq_slot, heads, dim, rd, rank, dense=None):
+                   page_size, tok_pos, tok_seq, seq_slot, heads, dim, rd, rank, dense=None, half_layout=False):
     """From the float32 projections of a latent attention layer: the cache row of every token
     (RMS-normed latent ``kv_in[:, :rank]``, then the key part ``kv_in[:, rank:]`` with its first
-    ``rot`` dims rotated as interleaved pairs) into the paged ``cache`` [pages, page_size, rank + rd];
+    ``rot`` dims rotated, as interleaved pairs or with ``half_layout`` as pairs (i, i + rot/2)) into the paged ``cache`` [pages, page_size, rank + rd];
     the queries' unrotated dims times ``q_scale`` into ``q_nope`` [T, heads * dim], their rotated
     dims (rotated, scaled) into the last ``rd`` columns of each head of ``q_lat``
     [T, heads * (rank + rd)]; ``gate`` [T, heads] = sigmoid(g_in) (float32; None: no gate).  ``dense``
@@ -872,7 +891,7 @@ def latent_prepare(q_in, kv_in, g_in, norm_w, eps, inv_freq, rot, q_scale, q_nop
     f = _fn("latent_attention", "gb_latent_prepare",
             [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_float,
              c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
-             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p])
+             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p])
     if dense is not None:
         assert dense.dtype == q_lat.dtype and dense.shape == (t, rank + rd) and dense.stride(1) == 1
     _check(f(q_in.data_ptr(), q_in.stride(0), kv_in.data_ptr(), kv_in.stride(0), _ptr(g_in),
@@ -880,7 +899,7 @@ def latent_prepare(q_in, kv_in, g_in, norm_w, eps, inv_freq, rot, q_scale, q_nop
              q_nope.data_ptr(), q_nope.stride(0), q_lat.data_ptr(), q_lat.stride(0), _ptr(gate), _ptr(cache),
              dtype_code(q_lat.dtype), _ptr(page_table), page_table.shape[1] if page_table is not None else 1, page_size,
              tok_pos.data_ptr(), tok_seq.data_ptr(), seq_slot.data_ptr(), t, heads, dim, rd, rank, _ptr(dense),
-             dense.stride(0) if dense is not None else 0, _stream()),
+             dense.stride(0) if dense is not None else 0, 1 if half_layout else 0, _stream()),
            "latent_prepare", "elementwise", _nbytes(q_in, kv_in, q_nope) + t * (rank + 2 * rd) * q_lat.element_size())
 
 
@@ -920,8 +939,8 @@ def grouped_gemm(a, lda, a_gstride, a_rows, a_div, w, w_gstride, c, ldc, c_gstri
     """Many bfloat16 products C_g = A_g W_g^T of unequal row counts in one tensor-core launch (see
     csrc/grouped_gemm.cu): group g's rows are offsets[g]..offsets[g+1] (None: ``rows`` each), an A
     row is a_rows[i] // a_div (None: i), C is bfloat16 or float32 by its dtype; ``gated``: W_g stacks
-    gate rows over up rows and C = min(g, limit) * sigmoid(alpha g) * (clamp(u) + shift); ``gated`` 2:
-    no gate rows, C = gelu(A W_g^T) in the exact (erf) form."""
+    gate rows over up rows and C = min(g, limit) * sigmoid(alpha g) * (clamp(u) + shift); ``gated`` 2 / 3:
+    no gate rows, C = gelu(A W_g^T) in the exact (erf) form / relu(A W_g^T)^2."""
     _cuda(a, w, c, scale, scale_rows, offsets, a_rows)
     assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and c.dtype in (torch.bfloat16, torch.float32)
     f = _fn("grouped_gemm", "gb_grouped_gemm",
@@ -1062,11 +1081,16 @@ def latent_attention_units(compute: str, rank: int, rd: int, dim: int = 0, vd: i
 
 # --------------------------------------------------------------------------- routed feed-forward
 
-def moe_topk(z, bias, experts, top, has_gate=False, all_softmax=False):
+ROUTINGS = {"softmax_top": 0, "softmax_all": 1, "sigmoid": 2}
+
+
+def moe_topk(z, bias, experts, top, has_gate=False, routing="softmax_top", scale: float = 1.0):
     """(idx int32 [T, top], weights float32 [T, top], shared float32 [T] or None) from the router's
     logits z (float32 [T, experts (+ 1)]): each token's ``top`` largest z + bias (the lower index wins
-    a tie), the softmax over those alone (with ``all_softmax``: their shares of the softmax over all
-    experts, which do not add up to one), and with ``has_gate`` the sigmoid of column ``experts``."""
+    a tie), weighed by ``routing`` times ``scale``: "softmax_top" the softmax over those alone,
+    "softmax_all" their shares of the softmax over all experts, which do not add up to one; "sigmoid":
+    scores s = sigmoid(z), the ``top`` largest s + bias, each s over the sum of the chosen s (+ 1e-20).
+    With ``has_gate`` the sigmoid of column ``experts``."""
     _cuda(z, bias)
     t = z.shape[0]
     assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[1] >= experts + (1 if has_gate else 0)
@@ -1075,17 +1099,19 @@ def moe_topk(z, bias, experts, top, has_gate=False, all_softmax=False):
     wts = torch.empty((t, top), dtype=torch.float32, device=z.device)
     sg = torch.empty((t,), dtype=torch.float32, device=z.device) if has_gate else None
     f = _fn("moe", "gb_moe_topk_mode", [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                        c_int, c_int, c_void_p])
+                                        c_int, c_int, c_float, c_void_p])
     _check(f(z.data_ptr(), z.stride(0), _ptr(bias), idx.data_ptr(), wts.data_ptr(), _ptr(sg), t, experts, top,
-             1 if has_gate else 0, 1 if all_softmax else 0, _stream()), "moe_topk", "elementwise", _nbytes(z))
+             1 if has_gate else 0, ROUTINGS[routing], float(scale), _stream()), "moe_topk", "elementwise", _nbytes(z))
     return idx, wts, sg
 
 
 def moe_experts(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down, residual, limit, shared_limit, alpha,
-                shift):
+                shift, col_scale=None):
     """residual[t] += sum_k wts[t, k] * expert_{idx[t, k]}(h[t]) + sg[t] * shared(h[t]), token-major
     (two kernels: gate/up with the activation, then down).  w_gate_up [E, 2 ff, width] (gate rows,
-    then up rows), w_down [E, width, ff]; the shared expert's [2 ffs, width] and [width, ffs], or None."""
+    then up rows), w_down [E, width, ff]; the shared expert's [2 ffs, width] and [width, ffs], or None.
+    ``col_scale`` (float32 [width]) multiplies what is added."""
+    _check_col_scale(col_scale, h.shape[1])
     _cuda(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down, residual)
     t, width = h.shape
     e, ff2, _ = w_gate_up.shape
@@ -1106,16 +1132,19 @@ def moe_experts(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down,
            _nbytes(h, y) + t * slots * 2 * ff * width * h.element_size())
     rows = torch.empty((t, slots, width), dtype=torch.float32, device=h.device)
     f = _fn("moe", "gb_moe_down", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                   c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                                   c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
     _check(f(y.data_ptr(), dtype_code(h.dtype), idx.data_ptr(), wts.data_ptr(), _ptr(sg), w_down.data_ptr(),
-             _ptr(shared_down), rows.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, ff, ffs, top, _stream()),
+             _ptr(shared_down), rows.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, ff, ffs, top,
+             _ptr(col_scale), _stream()),
            "moe_down", "matmul", _nbytes(y) + 2 * _nbytes(rows) + 2 * t * width * 4 + t * slots * ff * width * h.element_size())
     count_launches(1)   # the kernel that adds a token's rows
 
 
-def moe_experts_plain(h, idx, wts, w_up, w_down, residual):
-    """residual[t] += sum_k wts[t, k] * down_{idx[t, k]} gelu(up_{idx[t, k]} h[t]) for experts without a
-    gate (exact GELU), token-major.  w_up [E, ff, width], w_down [E, width, ff]."""
+def moe_experts_plain(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None):
+    """residual[t] += sum_k wts[t, k] * down_{idx[t, k]} act(up_{idx[t, k]} h[t]) for experts without a
+    gate (``act`` one of PLAIN_ACTS), token-major.  w_up [E, ff, width], w_down [E, width, ff].
+    ``col_scale`` (float32 [width]) multiplies what is added."""
+    _check_col_scale(col_scale, h.shape[1])
     _cuda(h, idx, wts, w_up, w_down, residual)
     t, width = h.shape
     e, ff, _ = w_up.shape
@@ -1123,21 +1152,22 @@ def moe_experts_plain(h, idx, wts, w_up, w_down, residual):
     assert w_up.is_contiguous() and w_down.is_contiguous() and w_down.shape == (e, width, ff) and w_up.shape[2] == width
     assert w_up.dtype == h.dtype == w_down.dtype and residual.dtype == torch.float32 and residual.stride(1) == 1
     y = torch.empty((t, top, ff), dtype=h.dtype, device=h.device)
-    f = _fn("moe", "gb_moe_up", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    f = _fn("moe", "gb_moe_up", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
     _check(f(h.data_ptr(), h.stride(0), dtype_code(h.dtype), idx.data_ptr(), w_up.data_ptr(), y.data_ptr(), t, width, ff, top,
-             _stream()), "moe_up", "matmul", _nbytes(h, y) + t * top * ff * width * h.element_size())
+             PLAIN_ACTS[act], _stream()), "moe_up", "matmul", _nbytes(h, y) + t * top * ff * width * h.element_size())
     rows = torch.empty((t, top, width), dtype=torch.float32, device=h.device)
     f = _fn("moe", "gb_moe_down", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                   c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                                   c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
     _check(f(y.data_ptr(), dtype_code(h.dtype), idx.data_ptr(), wts.data_ptr(), None, w_down.data_ptr(), None,
-             rows.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, ff, 0, top, _stream()),
+             rows.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, ff, 0, top, _ptr(col_scale),
+             _stream()),
            "moe_down", "matmul", _nbytes(y) + 2 * _nbytes(rows) + 2 * t * width * 4 + t * top * ff * width * h.element_size())
     count_launches(1)   # the kernel that adds a token's rows
 
 
-def moe_experts_plain_grouped(h, idx, wts, w_up, w_down, residual):
+def moe_experts_plain_grouped(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None):
     """As moe_experts_plain for a step of many tokens: entries ordered by expert, two grouped
-    tensor-core products (up with the GELU in its epilogue, down scaled by the routing weights), a
+    tensor-core products (up with the activation in its epilogue, down scaled by the routing weights), a
     token's rows added into the residual in slot order."""
     _cuda(h, idx, wts, w_up, w_down, residual)
     t, width = h.shape
@@ -1152,19 +1182,21 @@ def moe_experts_plain_grouped(h, idx, wts, w_up, w_down, residual):
            "elementwise", 3 * entries * 4)
     y = torch.empty((entries, ff), dtype=torch.bfloat16, device=h.device)
     grouped_gemm(h, h.stride(0), 0, perm, top, w_up, ff * width, y, ff, 0, None, None, 0, 0, offsets, e, 0, entries,
-                 ff, width, gated=2, what="moe_up_tc", nbytes=_nbytes(w_up, y) + entries * width * 2)
+                 ff, width, gated=1 + PLAIN_ACTS[act], what="moe_up_tc", nbytes=_nbytes(w_up, y) + entries * width * 2)
     rows = torch.empty((entries, width), dtype=torch.float32, device=h.device)
     grouped_gemm(y, ff, 0, None, 1, w_down, width * ff, rows, width, 0, wts.view(-1), perm, 1, 0, offsets, e, 0, entries,
                  width, ff, what="moe_down_tc", nbytes=_nbytes(w_down, y, rows))
-    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p])
-    _check(f(rows.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _stream()),
+    _check_col_scale(col_scale, width)
+    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(f(rows.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _ptr(col_scale),
+             _stream()),
            "moe_combine", "elementwise", _nbytes(rows) + 2 * t * width * 4)
 
 
-def moe_experts_plain_tc(h, idx, wts, w_up, w_down, residual):
+def moe_experts_plain_tc(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None):
     """As moe_experts_plain_grouped for a prompt step, the two products on the tcgen05 kernel (the
     activations copied into an order in which every expert's rows start at a multiple of the
-    tile's tokens; the GELU and the routing weight in the first product's epilogue)."""
+    tile's tokens; the activation and the routing weight in the first product's epilogue)."""
     _cuda(h, idx, wts, w_up, w_down, residual)
     t, width = h.shape
     e, ff, _ = w_up.shape
@@ -1183,11 +1215,13 @@ def moe_experts_plain_tc(h, idx, wts, w_up, w_down, residual):
     _check(f(h.data_ptr(), h.stride(0), row_entry.data_ptr(), tile_expert.data_ptr(), wts.data_ptr(), xp.data_ptr(),
              scale.data_ptr(), rows, width, top, bn, _stream()), "moe_permute", "elementwise", 2 * entries * width * 2)
     y = torch.empty((rows, ff), dtype=torch.bfloat16, device=h.device)
-    gemm_tc_grouped(xp, w_up.view(e * ff, width), y, ff, e, tile_expert, scale, gelu=True)
+    gemm_tc_grouped(xp, w_up.view(e * ff, width), y, ff, e, tile_expert, scale, act=act)
     out = torch.empty((rows, width), dtype=torch.float32, device=h.device)
     gemm_tc_grouped(y, w_down.view(e * width, ff), out, width, e, tile_expert)
-    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p])
-    _check(f(out.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _stream()),
+    _check_col_scale(col_scale, width)
+    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(f(out.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _ptr(col_scale),
+             _stream()),
            "moe_combine", "elementwise", entries * width * 4 + 2 * t * width * 4)
 
 
@@ -1202,7 +1236,7 @@ def moe_grouped_usable(h, w_gate_up, w_down) -> bool:
 
 
 def moe_experts_grouped(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down, residual, limit, shared_limit,
-                        alpha, shift):
+                        alpha, shift, col_scale=None):
     """As moe_experts for a step of many tokens: the (token, slot) entries are ordered by expert on the
     device, each expert's rows run as one product of a grouped tensor-core launch (gate/up with the
     activation, then down scaled by the routing weights), a token's rows are added into the residual
@@ -1225,10 +1259,12 @@ def moe_experts_grouped(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shar
     rows = torch.empty((entries, width), dtype=torch.float32, device=h.device)
     grouped_gemm(y, ff, 0, None, 1, w_down, width * ff, rows, width, 0, wts.view(-1), perm, 1, 0, offsets, e, 0, entries,
                  width, ff, what="moe_down_tc", nbytes=_nbytes(w_down, y, rows))
-    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p])
-    _check(f(rows.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _stream()),
+    _check_col_scale(col_scale, width)
+    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(f(rows.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _ptr(col_scale),
+             _stream()),
            "moe_combine", "elementwise", _nbytes(rows) + 2 * t * width * 4)
-    _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, alpha, shift)
+    _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, alpha, shift, col_scale)
 
 
 MOE_TC_MIN_TOKENS = 256
@@ -1243,28 +1279,29 @@ def moe_tc_usable(h, w_gate_up, w_down) -> bool:
 
 
 def gemm_tc_grouped(x, w, y, n, experts, tile_expert, row_scale=None, gated=False, limit=0.0, alpha=0.0, shift=0.0,
-                    bn=MOE_TC_TILE, gelu=False):
+                    bn=MOE_TC_TILE, act=None):
     """The tcgen05 product over groups of rows: x [rows, K] holds the groups one after the other, each
     starting at a multiple of ``bn`` rows; w stacks the groups' matrices ([experts * n, K], or
     [experts * 2 n, K] gated); tile_expert names the group of every tile of ``bn`` rows (-1: none).
     y float32 [rows, n], or with ``gated`` bfloat16 [rows, n] = row_scale * act(gate, up), or with
-    ``gelu`` bfloat16 [rows, n] = row_scale * gelu(x w^T) (erf form, no gate rows)."""
+    ``act`` (one of PLAIN_ACTS) bfloat16 [rows, n] = row_scale * act(x w^T) (no gate rows)."""
     _cuda(x, w, y, tile_expert, row_scale)
     rows, k = x.shape
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.stride(1) == 1 and w.is_contiguous()
-    assert not (gated and gelu)
-    assert y.shape == (rows, n) and y.is_contiguous() and y.dtype == (torch.bfloat16 if gated or gelu else torch.float32)
+    assert not (gated and act)
+    assert y.shape == (rows, n) and y.is_contiguous() and y.dtype == (torch.bfloat16 if gated or act else torch.float32)
     assert tile_expert.dtype == torch.int32 and tile_expert.numel() == rows // bn and rows % bn == 0
     f = _fn("gemm_tc", "gb_gemm_tc_grouped",
             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_int, c_int, c_int, c_void_p,
-             c_void_p, c_float, c_float, c_float, c_void_p])
-    _check(f(x.data_ptr(), w.data_ptr(), y.data_ptr(), 3 if gated else (0 if gelu else 1), rows, n, k, x.stride(0), y.stride(0), bn,
-             sm_count(x.device), experts, tile_expert.data_ptr(), _ptr(row_scale), limit, alpha, shift, _stream()),
+             c_void_p, c_float, c_float, c_float, c_int, c_void_p])
+    _check(f(x.data_ptr(), w.data_ptr(), y.data_ptr(), 3 if gated else (0 if act else 1), rows, n, k, x.stride(0), y.stride(0), bn,
+             sm_count(x.device), experts, tile_expert.data_ptr(), _ptr(row_scale), limit, alpha, shift, PLAIN_ACTS[act],
+             _stream()),
            "gemm_tc_grouped", "matmul", _nbytes(x, w, y))
 
 
 def moe_experts_tc(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down, residual, limit, shared_limit, alpha,
-                   shift):
+                   shift, col_scale=None):
     """As moe_experts_grouped for a prompt step, the experts' two products on the tcgen05 kernel: the
     activations are copied into an order in which every expert's rows start at a multiple of the
     tile's tokens (zeros between), the routing weight multiplies the activation's rows, and a token's
@@ -1291,13 +1328,15 @@ def moe_experts_tc(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_do
                     shift=shift)
     out = torch.empty((rows, width), dtype=torch.float32, device=h.device)
     gemm_tc_grouped(y, w_down.view(e * width, ff), out, width, e, tile_expert)
-    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p])
-    _check(f(out.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _stream()),
+    _check_col_scale(col_scale, width)
+    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(f(out.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _ptr(col_scale),
+             _stream()),
            "moe_combine", "elementwise", entries * width * 4 + 2 * t * width * 4)
-    _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, alpha, shift)
+    _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, alpha, shift, col_scale)
 
 
-def _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, alpha, shift):
+def _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, alpha, shift, col_scale=None):
     """residual += sg * shared(h): two dense products of the framework's around the activation."""
     if shared_down is None:
         return
@@ -1308,7 +1347,7 @@ def _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, a
     f = _fn("grouped_gemm", "gb_gated_act", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_void_p])
     _check(f(gu.data_ptr(), ys.data_ptr(), _ptr(sg), t, ffs, shared_limit, alpha, shift, _stream()), "gated_act",
            "elementwise", _nbytes(gu, ys))
-    gemm(ys, shared_down, residual, accumulate=True)
+    gemm(ys, shared_down, residual, accumulate=True, col_scale=col_scale)
 
 
 # --------------------------------------------------------------------------- sampling
@@ -1371,14 +1410,16 @@ def gemm_units(compute: str):
 NORM_LINKS = True
 
 
-def gemm(x, w, out, bias=None, accumulate=False, then_norm=None):
+def gemm(x, w, out, bias=None, accumulate=False, then_norm=None, act=None, col_scale=None):
     """out = x @ w.T (+ bias) or, with ``accumulate``, out += ...; picks the kernel for the
     precision and the shape: float32 runs on the CUDA cores in a fixed order; bfloat16 runs on the
     tensor cores, except for operands whose rows TMA cannot address (an inner size that is not
     a multiple of 8), which the plain kernel takes.  ``x`` may be UnscaledRows (a norm taken into
     this product).  ``then_norm`` = (weight, eps) of an RMSNorm that follows an accumulating
     product: where the kernel can, it leaves that norm's input as UnscaledRows, which is returned
-    (None: the norm has to run by itself)."""
+    (None: the norm has to run by itself).  ``act`` (one of PLAIN_ACTS): an activation of the results,
+    in the product's epilogue, before they are rounded.  ``col_scale`` (float32 [N]): with
+    ``accumulate``, multiplies what is added, per output feature."""
     link = x if isinstance(x, UnscaledRows) else None
     if link is not None:
         if norm_link_usable(link.rows, w, link.rows.shape[0]):
@@ -1388,12 +1429,12 @@ def gemm(x, w, out, bias=None, accumulate=False, then_norm=None):
     if x.dtype == torch.bfloat16 and gemm_tc_usable(x, w):
         m, n, k = x.shape[0], w.shape[0], x.shape[1]
         if m > 64:
-            gemm_tc_persistent(x, w, out, bias, accumulate)
+            gemm_tc_persistent(x, w, out, bias, accumulate, plain_act=act, col_scale=col_scale)
             return None
         if then_norm is not None and not (accumulate and gemm_tc_tiling(m, n, k)[1] >= 2):
             then_norm = None
-        return gemm_tc(x, w, out, bias, accumulate, link_in=link, link_out=then_norm)
-    gemm_ref(x, w, out, bias, accumulate)
+        return gemm_tc(x, w, out, bias, accumulate, link_in=link, link_out=then_norm, plain_act=act, col_scale=col_scale)
+    gemm_ref(x, w, out, bias, accumulate, act, col_scale)
     return None
 
 
@@ -1495,6 +1536,52 @@ def scale_rows(y: torch.Tensor, s: float):
     assert y.dtype == torch.float32 and y.is_contiguous()
     f = _fn("rows", "gb_scale_f32", [c_void_p, c_longlong, c_float, c_void_p])
     _check(f(y.data_ptr(), y.numel(), s, _stream()), "scale_rows", "elementwise", 2 * _nbytes(y))
+
+
+def cap_rows(y: torch.Tensor, cap: float):
+    """y = cap * tanh(y / cap) in place (float32)."""
+    _cuda(y)
+    assert y.dtype == torch.float32 and y.is_contiguous()
+    f = _fn("rows", "gb_cap_f32", [c_void_p, c_longlong, c_float, c_void_p])
+    _check(f(y.data_ptr(), y.numel(), cap, _stream()), "cap_rows", "elementwise", 2 * _nbytes(y))
+
+
+def embed_norm(table: torch.Tensor, tokens: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, scale: float, eps: float):
+    """out[t] = rmsnorm(table[tokens[t]] * scale) * weight; out is the float32 residual stream [T, H]."""
+    _cuda(table, tokens, weight, out)
+    assert tokens.dtype == torch.int32 and out.dtype == torch.float32 and out.is_contiguous() and table.is_contiguous()
+    assert weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == table.shape[1] == out.shape[1]
+    f = _fn("rows", "gb_embed_norm", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float,
+                                      c_void_p])
+    _check(f(table.data_ptr(), dtype_code(table.dtype), tokens.data_ptr(), weight.data_ptr(), out.data_ptr(), tokens.numel(),
+             table.shape[1], table.shape[0], scale, eps, _stream()), "embed_norm", "embed",
+           _nbytes(out) + tokens.numel() * table.shape[1] * table.element_size())
+
+
+def add_row(v: torch.Tensor, x: torch.Tensor, then=None):
+    """x[t] += v for every row of the float32 residual stream.  ``then`` = (weight, eps, out): the norm
+    that reads the stream next, taken in the same pass: out[t] = rmsnorm(x[t]) * weight."""
+    weight, eps, out = then if then is not None else (None, 0.0, None)
+    _cuda(v, x, weight, out)
+    n = x.shape[-1]
+    assert v.dtype == torch.float32 and v.is_contiguous() and v.numel() == n and x.dtype == torch.float32 and x.is_contiguous()
+    if then is not None:
+        assert weight.dtype == torch.float32 and weight.numel() == n and out.is_contiguous() and out.shape == x.shape
+    f = _fn("rows", "gb_add_row_norm", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p])
+    _check(f(v.data_ptr(), x.data_ptr(), x.numel() // n, n, _ptr(weight), _ptr(out),
+             dtype_code(out.dtype) if out is not None else F32, eps, _stream()), "add_row", "norm", 2 * _nbytes(x) + _nbytes(out))
+
+
+def norm_cols(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float):
+    """out[t] = rmsnorm(x[t]) * weight for a slice of columns ``x`` [T, n] of a float32 tensor."""
+    _cuda(x, weight, out)
+    xp, ldx = _cols(x)
+    t, n = x.shape
+    assert x.dtype == torch.float32 and weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == n
+    assert out.shape == (t, n) and out.is_contiguous()
+    f = _fn("rows", "gb_norm_cols", [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
+    _check(f(xp, ldx, weight.data_ptr(), out.data_ptr(), dtype_code(out.dtype), t, n, eps, _stream()), "norm_cols", "norm",
+           _nbytes(x, out))
 
 
 # --------------------------------------------------------------------------- mixers with a state per sequence
@@ -1732,6 +1819,39 @@ def wkv_scan(r, k, w, v, bonus, state, cu_seqlens, seq_slot, y, heads, dim, vdim
            _nbytes(y) * 5 + 2 * seq_slot.numel() * heads * dim * vdim * 4)
 
 
+def matrix_memory_aux_floats(dims: int, vdim: int) -> int:
+    """Floats per head that ``matrix_memory`` keeps for the vector n and the running maximum m: a set
+    for every 32 columns of the state, each padded as the state's dims are, m after n."""
+    lanes = 1 if dims <= 32 else (2 if dims <= 64 else (4 if dims <= 128 else 8))
+    return -(-vdim // 32) * (32 * lanes + 4)
+
+
+def matrix_memory(q, k, v, in_logit, forget_logit, state, aux, cu_seqlens, seq_slot, y, heads, dim, vdim, cap, q_scale):
+    """Matrix memory with exponential gates over each sequence of the packed step (float32 throughout):
+    i = cap tanh(in_logit / cap), f = logsigmoid(cap tanh(forget_logit / cap)) (cap 0: uncapped);
+    m' = max(f + m, i); S <- e^(f + m - m') S + e^(i - m') k v^T; n the same with k alone;
+    y = S^T q / (max(|n . q|, e^(-m')) + 1e-6), q times ``q_scale``.  All inputs are slices of columns of
+    one [T, *] tensor, q and k [T, heads * dim], v [T, heads * vdim], the logits [T, heads].  ``state``
+    [slots + 1, heads, recurrent_state_floats(dim, vdim)], ``aux`` [slots + 1, heads,
+    matrix_memory_aux_floats(dim, vdim)], both zeros for a new sequence; dim up to 256."""
+    _cuda(q, k, v, in_logit, forget_logit, state, aux, cu_seqlens, seq_slot, y)
+    for t in (q, k, v, in_logit, forget_logit, state, aux, y):
+        assert t.dtype == torch.float32
+    cols = [_cols(t) for t in (q, k, v, in_logit, forget_logit)]
+    ld = cols[0][1]
+    assert all(c[1] == ld for c in cols) and y.is_contiguous() and y.shape[1] == heads * vdim
+    assert q.shape[1] == k.shape[1] == heads * dim and v.shape[1] == heads * vdim
+    assert in_logit.shape[1] == forget_logit.shape[1] == heads
+    assert state.is_contiguous() and tuple(state.shape[1:]) == (heads, recurrent_state_floats(dim, vdim))
+    assert aux.is_contiguous() and tuple(aux.shape[1:]) == (heads, matrix_memory_aux_floats(dim, vdim))
+    f = _fn("recurrent", "gb_matrix_memory",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+             c_int, c_int, c_int, c_float, c_float, c_void_p])
+    _check(f(*[c[0] for c in cols], ld, state.data_ptr(), aux.data_ptr(), cu_seqlens.data_ptr(), seq_slot.data_ptr(), y.data_ptr(),
+             seq_slot.numel(), heads, dim, vdim, float(cap or 0.0), q_scale, _stream()), "matrix_memory", "attention",
+           _nbytes(q, k, v, y) + 2 * seq_slot.numel() * heads * dim * vdim * 4)
+
+
 # --------------------------------------------------------------------------- attention with capped scores
 
 def filter_rope_cache(u, taps, state, inv_freq, rot, ctx_pos, tok_seq, seq_slot, cu_seqlens, page_table, page_size, q_out,
@@ -1792,12 +1912,13 @@ def attention_capped_units(compute: str, dim: int, vdim: int, page_size: int = 6
 
 
 def attention_capped(ctx, q, out, heads, kcache, vcache, page_table, page_size, window, scale, cap, gate=None,
-                     out_scale: float = 1.0, keep_first: int = 0, sink=None):
+                     out_scale: float = 1.0, keep_first: int = 0, sink=None, gate_per_head: bool = False):
     """Attention of the step's queries [T, heads * dim] over the cache with keys of ``dim`` and
     values of ``vdim``: score = (q . k) * scale, capped as cap * tanh(score / cap) when ``cap``;
     a window of ``window`` keys when given, beside which the first ``keep_first`` keys of the
     sequence stay visible; ``sink`` (float32 [heads]): exp(sink[head]) is one more term of the
-    softmax's denominator; the output times sigmoid(gate) * out_scale.  bfloat16
+    softmax's denominator; the output times sigmoid(gate) * out_scale, ``gate`` [T, heads * vdim] or with
+    ``gate_per_head`` [T, heads].  bfloat16
     steps run on the tensor cores where the sizes allow (keys a multiple of 16, values of 8, up to
     256), prompts and single tokens alike; float32 and other sizes run the plain kernel."""
     _cuda(q, out, kcache, vcache, page_table, gate, sink)
@@ -1809,24 +1930,25 @@ def attention_capped(ctx, q, out, heads, kcache, vcache, page_table, page_size, 
     gp, ldg = _cols(gate) if gate is not None else (None, 0)
     assert q.dtype == out.dtype == kcache.dtype == vcache.dtype and (gate is None or gate.dtype == q.dtype)
     assert q.shape[1] == heads * dim and out.shape[1] == heads * vdim
+    assert gate is None or gate.shape[1] >= (heads if gate_per_head else heads * vdim)
     if (CAPPED_ATTENTION_MMA and attention_capped_mma_usable(q.dtype, dim, vdim, page_size)
             and getattr(ctx, "cu_seqlens", None) is not None and qp % 16 == 0 and ldq % 8 == 0 and op % 4 == 0
-            and ldo % 2 == 0 and (gp or 0) % 4 == 0 and ldg % 2 == 0):
+            and ldo % 2 == 0 and (gate_per_head or ((gp or 0) % 4 == 0 and ldg % 2 == 0))):
         f = _fn("attention_capped_mma", "gb_attention_capped_mma",
                 [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_float, c_void_p,
-                 c_longlong, c_float, c_int, c_void_p], (("GB_HEAD_DIM", dim), ("GB_VALUE_DIM", vdim)))
+                 c_longlong, c_float, c_int, c_int, c_void_p], (("GB_HEAD_DIM", dim), ("GB_VALUE_DIM", vdim)))
         _check(f(qp, ldq, op, ldo, kcache.data_ptr(), vcache.data_ptr(), page_table.data_ptr(), page_table.shape[1], page_size,
                  groups, dim, vdim, ctx.cu_seqlens.data_ptr(), ctx.seq_start.data_ptr(), ctx.seq_slot.data_ptr(), ctx.n_seqs,
                  q.shape[0], heads, int(window or 0), keep_first, _ptr(sink), scale, float(cap or 0.0), gp, ldg, out_scale,
-                 1 if q.shape[0] == ctx.n_seqs else 0, _stream()),
+                 1 if gate_per_head else 0, 1 if q.shape[0] == ctx.n_seqs else 0, _stream()),
                "attention_capped_mma", "attention", 2 * q.numel() * q.element_size())
         return
     f = _fn("attention_capped", "gb_attention_capped",
             [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_float, c_void_p, c_longlong, c_float,
-             c_void_p])
+             c_int, c_void_p])
     _check(f(qp, ldq, op, ldo, dtype_code(q.dtype), kcache.data_ptr(), vcache.data_ptr(), page_table.data_ptr(),
              page_table.shape[1], page_size, groups, dim, vdim, ctx.tok_pos.data_ptr(), ctx.tok_seq.data_ptr(),
              ctx.seq_slot.data_ptr(), q.shape[0], heads, int(window or 0), keep_first, _ptr(sink), scale, float(cap or 0.0),
-             gp, ldg, out_scale, _stream()), "attention_capped", "attention", 2 * q.numel() * q.element_size())
+             gp, ldg, out_scale, 1 if gate_per_head else 0, _stream()), "attention_capped", "attention", 2 * q.numel() * q.element_size())

@@ -26,6 +26,10 @@ Interfaces (all tensors on the device; ``ctx`` is the ``StepContext`` of the run
   kind); ``parts()`` -> {name: part}, every part it built; ``forward(ctx, x, caches,
   writes_cache)`` runs them on ``x`` in place, ``caches`` being the views of all its parts'
   needs in the order of ``parts()`` (``Block.split_caches`` deals them out).
+* scale: ``factor()`` -> float32 [hidden], a factor per feature on what a mixer or feed-forward adds; the
+  block hands it to the part's ``set_output_scale`` once both are loaded.
+* stream: ``forward(ctx, x, then_norm=None)`` changes the residual stream between two runs of layers
+  (``ScheduleEntry.before``) and returns ``then_norm``'s output when it made it in the same pass.
 * embedding: ``forward(ctx, tokens, out)``; head: ``forward(ctx, h)`` -> float32 logits.
 
 Optional, for decode steps: a norm taken into the products around it.  A mixer or feed-forward
@@ -164,7 +168,7 @@ class Block(Part):
 
 
 _REGISTRY: Dict[Tuple[str, str], Callable] = {}
-CATEGORIES = ("norm", "position", "mixer", "ffn", "block", "embedding", "head")
+CATEGORIES = ("norm", "position", "mixer", "ffn", "block", "scale", "stream", "embedding", "head")
 
 
 def register_part(category: str, kind: str, factory: Callable) -> None:

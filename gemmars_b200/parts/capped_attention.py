@@ -26,7 +26,8 @@ its key head as projected (with its bias), before norm and rotation, so vdim == 
 its dims (``q_norm``, ``k_norm``, shared by the heads) before the rotation.  ``q_temper`` {"coef",
 "every"}: the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
 ``fixed_sink`` (a number s): exp(s) joins the softmax's denominator for every head, without a
-tensor (0.0: one is added to the denominator).
+tensor (0.0: one is added to the denominator).  ``gate`` may be "head": one number per head,
+sigmoid(W_g h)[head], instead of one per output channel.
 Parameters: hidden_size, heads, kv_heads, dim, vdim, bias, conv, window, keep_first, sink, scale,
 softcap, gate, position, has_kv, ring, out_scale, values_are_keys, qk_norm, q_temper, fixed_sink.
 """
@@ -51,6 +52,9 @@ class CappedAttention(Part):
         self.heads, self.kv_heads = int(p["heads"]), int(p["kv_heads"])
         self.dim, self.vdim = int(p["dim"]), int(p["vdim"])
         self.bias, self.gate = bool(p.get("bias", False)), bool(p.get("gate", False))
+        if p.get("gate") not in (None, False, True, "head"):
+            raise ValueError(f"capped_attention: gate must be a truth value or 'head', got {p.get('gate')!r}")
+        self.gate_per_head = p.get("gate") == "head"
         self.taps = int(p.get("conv") or 0)
         self.window = p.get("window")
         self.keep_first = int(p.get("keep_first") or 0)
@@ -111,7 +115,7 @@ class CappedAttention(Part):
             if self.has_kv:
                 w["k_norm"] = TensorWant((d,), "vector")
         if self.gate:
-            w["g"] = TensorWant((nh * vd, h))
+            w["g"] = TensorWant((nh if self.gate_per_head else nh * vd, h))
         if self.sink:
             w["sink"] = TensorWant((nh,), "vector")
         return w
@@ -123,9 +127,9 @@ class CappedAttention(Part):
         if self.bias:
             parts = [t[n + "_bias"] for n in qkv]
             if self.gate:
-                parts.append(torch.zeros(self.heads * self.vdim, dtype=torch.float32, device=t["q_bias"].device))
+                parts.append(torch.zeros(t["g"].shape[0], dtype=torch.float32, device=t["q_bias"].device))
             bias = torch.cat(parts)
-        self.proj = Linear(torch.cat([t[n] for n in names], dim=0), bias)     # one product: [q | k | v | gate]
+        self.proj = Linear.stacked([t[n] for n in names], bias, 8 if self.gate_per_head else 1)   # one product: [q | k | v | gate]
         self.o = Linear(t["o"])
         if self.taps:
             self.filter = torch.cat([t[n + "_conv"] for n in qkv], dim=0).contiguous()
@@ -136,6 +140,13 @@ class CappedAttention(Part):
         if self.qk_norm_eps is not None:
             self.q_norm = t["q_norm"].to(torch.float32).contiguous()
             self.k_norm = t["k_norm"].to(torch.float32).contiguous() if self.has_kv else None
+
+    #: forward takes ``then_norm`` and may be given kernels.UnscaledRows for ``h``
+    links_norms = True
+
+    def set_output_scale(self, scale):
+        """``scale`` (float32 [hidden]) multiplies what the mixer adds."""
+        self.o.out_scale = scale
 
     def kernel_units(self):
         return (kernels.gemm_units(self.compute) + kernels.attention_capped_units(self.compute, self.dim, self.vdim)
@@ -152,7 +163,7 @@ class CappedAttention(Part):
     def weight_bytes(self):
         return self.proj.bytes() + self.o.bytes() + (4 * self.filter.numel() if self.filter is not None else 0)
 
-    def forward(self, ctx, h, residual, caches, writes_cache=True):
+    def forward(self, ctx, h, residual, caches, writes_cache=True, then_norm=None):
         if writes_cache != self.has_kv:
             raise ValueError("capped_attention: a part with keys and values of its own writes its own cache, and one "
                              "without reads another entry's (has_kv and the schedule's cache_of must agree)")
@@ -179,8 +190,9 @@ class CappedAttention(Part):
             kernels.short_filter_state(p[:, :c], filter_state, ctx.cu_seqlens, ctx.seq_slot, self.taps)
         att = torch.empty((t, nh * vd), dtype=p.dtype, device=p.device)
         kernels.attention_capped(ctx, q, att, nh, kc, vc, group.page_table, group.page_size, self.window, self.scale,
-                                 self.softcap, p[:, c:] if self.gate else None, self.out_scale, self.keep_first, self.sinks)
-        self.o.add_into(att, residual)
+                                 self.softcap, p[:, c:] if self.gate else None, self.out_scale, self.keep_first, self.sinks,
+                                 self.gate_per_head)
+        return self.o.add_into(att, residual, then_norm)
 
 
 register_part("mixer", "capped_attention", CappedAttention)

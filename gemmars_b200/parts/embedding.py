@@ -7,7 +7,10 @@ src/qwen.rs:472-485).
 
 ``positions`` (embedding, default none): rows of a second table, a learned vector per position
 that is added to the token's row unscaled, x[t] += P[position of t]; a sequence cannot grow
-beyond the table.  ``logit_scale`` (head, default 1): the float32 logits are multiplied by it."""
+beyond the table.  ``norm`` (embedding, default none) {"eps", "scalar"}: the token's row passes an
+RMSNorm before it becomes the stream, its weight a vector or with ``scalar`` one number.
+``logit_scale`` (head, default 1): the float32 logits are multiplied by it; ``logit_softcap`` (head,
+default none): they become cap * tanh(logits / cap)."""
 from __future__ import annotations
 
 import torch
@@ -26,24 +29,34 @@ class Embedding(Part):
         self.hidden_size = int(spec.params["hidden_size"])
         self.scale = spec.params.get("scale") or 1.0
         self.n_positions = int(spec.params.get("positions") or 0)
-        self.table = self.positions = None
+        norm = spec.params.get("norm")
+        self.norm_eps = float(norm["eps"]) if norm else None
+        self.norm_scalar = bool(norm.get("scalar", False)) if norm else False
+        self.table = self.positions = self.norm_weight = None
 
     def wants(self):
         w = {"weight": TensorWant((self.vocab_size, self.hidden_size), "matrix")}
         if self.n_positions:
             w["positions"] = TensorWant((self.n_positions, self.hidden_size), "matrix")
+        if self.norm_eps is not None:
+            w["norm"] = TensorWant(() if self.norm_scalar else (self.hidden_size,), "vector")
         return w
 
     def load(self, tensors):
         self.table = tensors["weight"].contiguous()
         if self.n_positions:
             self.positions = tensors["positions"].contiguous()
+        if self.norm_eps is not None:
+            self.norm_weight = tensors["norm"].to(torch.float32).reshape(-1).expand(self.hidden_size).contiguous()
 
     def kernel_units(self):
-        return [("elementwise", ())] + ([("rows", ())] if self.n_positions else [])
+        return [("elementwise", ())] + ([("rows", ())] if self.n_positions or self.norm_eps is not None else [])
 
     def forward(self, ctx, tokens, out):
-        kernels.embed_gather(self.table, tokens, out, float(self.scale))
+        if self.norm_eps is not None:
+            kernels.embed_norm(self.table, tokens, self.norm_weight, out, float(self.scale), self.norm_eps)
+        else:
+            kernels.embed_gather(self.table, tokens, out, float(self.scale))
         if self.n_positions:
             if ctx.max_total > self.n_positions and ctx.pad_slot is None:
                 raise ValueError(f"a sequence of {ctx.max_total} tokens is longer than the position table "
@@ -59,6 +72,7 @@ class LinearHead(Part):
         self.vocab_size = int(spec.params["vocab_size"])
         self.hidden_size = int(spec.params["hidden_size"])
         self.logit_scale = float(spec.params.get("logit_scale") or 1.0)
+        self.softcap = float(spec.params.get("logit_softcap") or 0.0)
         self.proj = None
 
     def wants(self):
@@ -68,13 +82,15 @@ class LinearHead(Part):
         self.proj = Linear(tensors["weight"])
 
     def kernel_units(self):
-        return kernels.gemm_units(self.compute) + ([("rows", ())] if self.logit_scale != 1.0 else [])
+        return kernels.gemm_units(self.compute) + ([("rows", ())] if self.logit_scale != 1.0 or self.softcap else [])
 
     def forward(self, ctx, h):
         with kernels.profile_category("lm_head"):
             logits = self.proj(h, out_dtype=torch.float32)
             if self.logit_scale != 1.0:
                 kernels.scale_rows(logits, self.logit_scale)
+            if self.softcap:
+                kernels.cap_rows(logits, self.softcap)
             return logits
 
     def weight_bytes(self):

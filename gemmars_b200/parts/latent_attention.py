@@ -17,9 +17,12 @@ the query (q_nope[h] . Wuk[h] c = (Wuk[h]^T q_nope[h]) . c) and Wuv[h] to the at
 over the latents (sum_j p_j Wuv[h] c_j = Wuv[h] sum_j p_j c_j), so prompts, continued prompts and
 single tokens all run one attention kernel over the cached rows, with all heads sharing them.
 
+With ``q_rank`` the queries pass a latent of their own: q = Wuq (rmsnorm(Wdq h) * w_q).
+
 All sizes and constants are parameters: hidden_size, num_heads, dim, rot_dim, vdim, rank, scale,
-norm_eps, gate (whether the output gate exists), window (None: all keys), position (a PartSpec of
-kind ``rotary`` with the interleaved layout, or None).
+norm_eps, gate (whether the output gate exists), window (None: all keys), q_rank (None: queries straight
+from h), position (a PartSpec of kind ``rotary``, of either layout, or None), out_scale (a factor on the
+result, applied in float32 after the output product).
 """
 from __future__ import annotations
 
@@ -51,39 +54,66 @@ class LatentAttention(Part):
         pos = p.get("position")
         self.position = build_part("position", pos, compute) if pos is not None else None
         if self.position is not None:
-            if not isinstance(self.position, Rotary) or self.position.layout != "interleaved":
-                raise ValueError("latent_attention: the kernel that writes the cache rows rotates interleaved pairs; "
-                                 "its position encoding must be a rotary part with that layout, or none")
+            if not isinstance(self.position, Rotary) or self.position.magnitude != 1.0:
+                raise ValueError("latent_attention: the position encoding must be a rotary part without a magnitude, or none")
             if self.position.rotary_dim > self.rot_dim:
                 raise ValueError(f"latent_attention: cannot rotate {self.position.rotary_dim} of {self.rot_dim} dims")
         if min(self.num_heads, self.rank, self.vdim) <= 0 or self.dim < 0 or self.rot_dim < 0 or self.dim + self.rot_dim <= 0:
             raise ValueError("latent_attention: heads, rank and vdim must be positive, and a head must have query dims")
-        self.proj = self.o = self.uk_t = self.uv = self.norm_w = None
+        self.q_rank = int(p["q_rank"]) if p.get("q_rank") is not None else None
+        if self.q_rank is not None and self.q_rank < 1:
+            raise ValueError(f"latent_attention: q_rank must be positive, got {self.q_rank}")
+        self.out_scale = float(p.get("out_scale", 1.0))
+        self.proj = self.uq = self.o = self.uk_t = self.uv = self.norm_w = self.q_norm_w = None
 
     # ---- weights
     def wants(self):
         h, nh, r = self.hidden_size, self.num_heads, self.rank
-        w = {"q": TensorWant((nh * (self.dim + self.rot_dim), h)), "dkv": TensorWant((r + self.rot_dim, h)),
-             "dkv_norm": TensorWant((r,), "vector"), "uk": TensorWant((nh * self.dim, r)),
-             "uv": TensorWant((nh * self.vdim, r)), "o": TensorWant((h, nh * self.vdim))}
+        qd = nh * (self.dim + self.rot_dim)
+        if self.q_rank is None:
+            w = {"q": TensorWant((qd, h))}
+        else:
+            w = {"dq": TensorWant((self.q_rank, h)), "dq_norm": TensorWant((self.q_rank,), "vector"),
+                 "uq": TensorWant((qd, self.q_rank))}
+        w.update({"dkv": TensorWant((r + self.rot_dim, h)), "dkv_norm": TensorWant((r,), "vector"),
+                  "uk": TensorWant((nh * self.dim, r)), "uv": TensorWant((nh * self.vdim, r)),
+                  "o": TensorWant((h, nh * self.vdim))})
         if self.gated:
             w["g"] = TensorWant((nh, h))
         return w
 
     def load(self, t):
         nh, r = self.num_heads, self.rank
-        # one product reads the input once: queries, then the latent and the key part, then the gate logits
-        self.proj = Linear(torch.cat([t["q"], t["dkv"]] + ([t["g"]] if self.gated else []), dim=0))
+        # one product reads the input once: queries (or their latent), then the latent and the key part,
+        # then the gate logits
+        first = t["q"] if self.q_rank is None else t["dq"]
+        self.proj = Linear.stacked([first, t["dkv"]] + ([t["g"]] if self.gated else []),
+                                   multiple=1 if self.q_rank is None else 4)
+        if self.q_rank is not None:
+            self.uq, self.q_norm_w = Linear(t["uq"]), t["dq_norm"].contiguous()
         self.o = Linear(t["o"])
+        if self.out_scale != 1.0:
+            self.set_output_scale(None)
         # [heads, rank, dim]: the matrix that carries a head's unrotated query dims into the latent space
         self.uk_t = t["uk"].view(nh, self.dim, r).transpose(1, 2).contiguous()
         self.uv = t["uv"].view(nh, self.vdim, r).contiguous()
         self.uk = t["uk"].view(nh, self.dim, r).contiguous()     # as stored: for prompts that expand the keys
         self.norm_w = t["dkv_norm"].contiguous()
 
+    #: forward takes ``then_norm`` and may be given kernels.UnscaledRows for ``h``
+    links_norms = True
+
+    def set_output_scale(self, scale):
+        """``scale`` (float32 [hidden], None: ones) multiplies what the mixer adds, beside ``out_scale``."""
+        if scale is None:
+            scale = torch.ones(self.hidden_size, dtype=torch.float32, device=self.o.weight.device)
+        self.o.out_scale = scale * self.out_scale
+
     def kernel_units(self):
         units = kernels.gemm_units(self.compute) + kernels.latent_attention_units(self.compute, self.rank, self.rot_dim,
                                                                                   self.dim, self.vdim)
+        if self.q_rank is not None:
+            units = units + [("rows", ())]
         return units + ([("grouped_gemm", ())] if self.compute != "float32" else [])
 
     def cache_needs(self):
@@ -91,15 +121,22 @@ class LatentAttention(Part):
 
     def weight_bytes(self):
         per = self.uk_t.element_size()     # a decode step reads the transposed copy, not self.uk
-        return self.proj.bytes() + self.o.bytes() + (self.uk_t.numel() + self.uv.numel()) * per + 4 * self.norm_w.numel()
+        queries = self.uq.bytes() + 4 * self.q_rank if self.q_rank is not None else 0
+        return self.proj.bytes() + queries + self.o.bytes() + (self.uk_t.numel() + self.uv.numel()) * per + 4 * self.norm_w.numel()
 
     # ---- step
-    def forward(self, ctx, h, residual, caches, writes_cache=True):
+    def forward(self, ctx, h, residual, caches, writes_cache=True, then_norm=None):
         nh, dim, rd, r, vd = self.num_heads, self.dim, self.rot_dim, self.rank, self.vdim
         group, kc, _ = caches[0]
         t = h.shape[0]
-        nq = nh * (dim + rd)
+        nq = nh * (dim + rd) if self.q_rank is None else self.q_rank
         proj = self.proj(h, out_dtype=torch.float32)          # norms, angles and the gate are float32 work
+        h = h.rows if isinstance(h, kernels.UnscaledRows) else h
+        q = proj[:, :nq]
+        if self.q_rank is not None:
+            cq = torch.empty((t, nq), dtype=self.act_dtype, device=h.device)
+            kernels.norm_cols(q, self.q_norm_w, cq, self.eps)
+            q = self.uq(cq, out_dtype=torch.float32)
         q_nope = torch.empty((t, nh * dim), dtype=self.act_dtype, device=h.device)
         qa = torch.empty((t, nh * (r + rd)), dtype=self.act_dtype, device=h.device)
         gate = torch.empty((t, nh), dtype=torch.float32, device=h.device) if self.gated else None
@@ -109,11 +146,11 @@ class LatentAttention(Part):
         expand = (self.window is None and t >= kernels.LATENT_EXPAND_MIN_TOKENS and ctx.host is not None
                   and not any(ctx.host["seq_start"]) and kernels.latent_expand_usable(h.dtype, r, dim, rd, vd))
         dense = torch.empty((t, r + rd), dtype=self.act_dtype, device=h.device) if expand else None
-        kernels.latent_prepare(proj[:, :nq], proj[:, nq:nq + r + rd], proj[:, nq + r + rd:] if self.gated else None,
+        kernels.latent_prepare(q, proj[:, nq:nq + r + rd], proj[:, nq + r + rd:nq + r + rd + nh] if self.gated else None,
                                self.norm_w, self.eps, self.position.inv_freq(h.device) if rot else None, rot, self.scale,
                                q_nope, qa, gate, kc.view(-1, group.page_size, r + rd) if writes_cache else None,
                                group.page_table, group.page_size, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, nh, dim, rd, r,
-                               dense=dense)
+                               dense=dense, half_layout=self.position is not None and self.position.layout == "half")
         if expand:
             return self._expanded(ctx, q_nope, qa, gate, dense, residual)
         if dim:
@@ -125,8 +162,7 @@ class LatentAttention(Part):
                                  group.page_size, self.window)
         o = torch.empty((t, nh * vd), dtype=self.act_dtype, device=h.device)
         kernels.heads_gemm(lat.view(t, nh, r), self.uv, o.view(t, nh, vd), nh, scale=gate)
-        self.o.add_into(o, residual)
-
+        return self.o.add_into(o, residual, then_norm)
 
     def _expanded(self, ctx, q_nope, qa, gate, dense, residual):
         """Attention of a prompt step over keys and values expanded per head.  Every head gets rows

@@ -13,11 +13,13 @@ hidden_size, experts, top, ff, limit, alpha (1.702), shift (1.0), router_bias, a
 a sigmoid of one number per token).  A ``limit`` of None clamps nothing; with alpha 1 and shift 0
 the expert is then the plain gated form silu(gate h) * (up h).
 
-Two more parameters.  ``gated`` False: an expert has no gate matrix, out = down gelu(up h) with the
-exact (erf) GELU (its tensors are ``e<j>.up`` and ``e<j>.down``; no clamps, no shared expert).
-``routing`` "softmax_all": the weights are the chosen experts' shares of the softmax over all
-experts, as they are (they do not add up to one); the default "softmax_top" is the softmax over the
-chosen alone.
+More parameters.  ``gated`` False: an expert has no gate matrix, out = down act(up h), ``activation``
+"gelu" (the exact, erf form; the default) or "relu2" (the square of relu); its tensors are ``e<j>.up``
+and ``e<j>.down``; no clamps, no shared expert.  ``routing`` "softmax_all": the weights are the chosen
+experts' shares of the softmax over all experts, as they are (they do not add up to one); "sigmoid":
+the scores are s = sigmoid(z), the ``top`` largest s + router_bias are chosen, and a chosen expert's
+weight is its s (without the bias) over the sum of the chosen s (+ 1e-20); the default "softmax_top"
+is the softmax over the chosen alone.  ``routing_scale`` (1) multiplies the weights.
 """
 from __future__ import annotations
 
@@ -44,8 +46,13 @@ class RoutedExperts(Part):
         self.router_bias = bool(p.get("router_bias", True))
         self.gated = bool(p.get("gated", True))
         self.routing = p.get("routing", "softmax_top")
-        if self.routing not in ("softmax_top", "softmax_all"):
-            raise ValueError(f"moe: unknown routing {self.routing!r} (softmax_top or softmax_all)")
+        if self.routing not in kernels.ROUTINGS:
+            raise ValueError(f"moe: unknown routing {self.routing!r} (known: {', '.join(kernels.ROUTINGS)})")
+        self.routing_scale = float(p.get("routing_scale", 1.0))
+        self.activation = p.get("activation", "gelu")
+        if not self.gated and (self.activation is None or self.activation not in kernels.PLAIN_ACTS):
+            raise ValueError(f"moe: activation {self.activation!r} has no kernel for experts without a gate")
+        self.out_scale = None
         if not self.gated and (p.get("shared") or p.get("limit") is not None):
             raise ValueError("moe: experts without a gate take no clamp and no shared expert")
         shared = p.get("shared")
@@ -97,7 +104,11 @@ class RoutedExperts(Part):
     def _route(self, h):
         z = self.router(h, out_dtype=torch.float32)
         return kernels.moe_topk(z, self.bias, self.experts, self.top, has_gate=bool(self.shared_ff and self.shared_gated),
-                                all_softmax=self.routing == "softmax_all")
+                                routing=self.routing, scale=self.routing_scale)
+
+    def set_output_scale(self, scale):
+        """``scale`` (float32 [hidden]) multiplies what the feed-forward adds."""
+        self.out_scale = scale
 
     def weight_bytes(self):
         """What a decode step of one token reads: the router, ``top`` experts, the shared expert."""
@@ -124,7 +135,7 @@ class RoutedExperts(Part):
                 run = kernels.moe_experts_plain_grouped
             else:
                 run = kernels.moe_experts_plain
-            run(h, idx, wts, self.gate_up, self.down, residual)
+            run(h, idx, wts, self.gate_up, self.down, residual, act=self.activation, col_scale=self.out_scale)
             return
         if self.shared_ff and sg is None:
             sg = torch.ones((h.shape[0],), dtype=torch.float32, device=h.device)
@@ -135,7 +146,7 @@ class RoutedExperts(Part):
         else:
             run = kernels.moe_experts
         run(h, idx, wts, sg, self.gate_up, self.down, self.shared_gate_up, self.shared_down, residual,
-                            self.limit, self.shared_limit, self.alpha, self.shift)
+            self.limit, self.shared_limit, self.alpha, self.shift, col_scale=self.out_scale)
 
 
 register_part("ffn", "moe", RoutedExperts)

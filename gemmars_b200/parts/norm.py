@@ -4,7 +4,8 @@ src/config.rs:465-469).  Input: rows of the float32 residual stream; output: act
 
 ``offset`` (default 0): the stored weight is a deviation from it, w = offset + stored (a
 checkpoint that keeps its norm weights around zero has offset 1); the sum is taken once, in
-float32, when the weight is loaded.  ``add_normed`` is the norm on the other side of a sublayer:
+float32, when the weight is loaded.  ``scalar`` (default False): the weight is one number for all
+coordinates (a tensor of shape []), spread over them when it is loaded.  ``add_normed`` is the norm on the other side of a sublayer:
 it norms the sublayer's float32 output and adds it into the residual stream.  ``forward_with`` is two
 norms of the same rows in one pass (a block whose mixer and feed-forward each read a norm of their
 own of the same x)."""
@@ -27,13 +28,16 @@ class RMSNorm(Part):
         self.size = int(spec.params["size"])
         self.eps = float(spec.params["eps"])
         self.offset = float(spec.params.get("offset", 0.0))
+        self.scalar = bool(spec.params.get("scalar", False))
         self.weight = None
 
     def wants(self):
-        return {"weight": TensorWant((self.size,), "vector")}
+        return {"weight": TensorWant(() if self.scalar else (self.size,), "vector")}
 
     def load(self, tensors):
         w = tensors["weight"].to(torch.float32)
+        if self.scalar:
+            w = w.reshape(1).expand(self.size)
         self.weight = (w + self.offset if self.offset else w).contiguous()
 
     def kernel_units(self):

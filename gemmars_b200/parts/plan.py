@@ -43,9 +43,11 @@ class LayerSpec:
 class ScheduleEntry:
     """One run of a layer.  A layer may be named by several entries; each entry that keeps a
     cache has storage of its own.  ``cache_of`` is the position in the schedule of an earlier
-    entry whose cache this run reads instead of writing one (None: its own)."""
+    entry whose cache this run reads instead of writing one (None: its own).  ``before``: a part of
+    category ``stream`` that changes the residual stream right before this run (None: nothing does)."""
     layer: int
     cache_of: Optional[int] = None
+    before: Optional[PartSpec] = None
 
 
 @dataclasses.dataclass

@@ -5,6 +5,8 @@ sum of theirs, each times a factor of its own.
 into the same float32 rows, in the order listed; the factor is handed to the branch as its
 ``out_scale`` parameter, which it applies in float32 before its output product.  Tensors, cache
 needs, kernels and weight bytes are the branches' own, its tensors under ``<name>.<short name>``.
+A factor per output feature (``set_output_scale``) is handed to every branch.  Where all branches can,
+a norm before the mixer is taken into their products, and the norm after it into the last branch's.
 """
 from __future__ import annotations
 
@@ -52,13 +54,26 @@ class SideBySide(Part):
     def capture_depends_on_length(self):
         return any(part.capture_depends_on_length for _, part in self.branches)
 
-    def forward(self, ctx, h, residual, caches, writes_cache=True):
-        at = 0
+    @property
+    def links_norms(self):
+        return all(getattr(part, "links_norms", False) for _, part in self.branches)
+
+    def set_output_scale(self, scale):
+        for name, part in self.branches:
+            if not hasattr(part, "set_output_scale"):
+                raise ValueError(f"side_by_side: branch {name!r} takes no factor on its output")
+            part.set_output_scale(scale)
+
+    def forward(self, ctx, h, residual, caches, writes_cache=True, then_norm=None):
+        at, left = 0, None
         caches = list(caches or [])
-        for _, part in self.branches:
+        last = len(self.branches) - 1
+        for i, (_, part) in enumerate(self.branches):
             n = len(part.cache_needs())
-            part.forward(ctx, h, residual, caches[at:at + n], writes_cache)
+            extra = {"then_norm": then_norm} if i == last and then_norm is not None else {}
+            left = part.forward(ctx, h, residual, caches[at:at + n], writes_cache, **extra)
             at += n
+        return left if then_norm is not None else None
 
 
 register_part("mixer", "side_by_side", SideBySide)
