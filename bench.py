@@ -2,7 +2,7 @@
 """Decode and prefill throughput of Qwen3-shaped models with random weights on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl reference] [--config 8b|4b|32b]
-    python bench.py --compare toretar|kuporax|dalerax|nogosun [--sizes small,lite,mid] [--batch 8] [--context 4096]
+    python bench.py --compare toretar|kuporax|dalerax|nogosun|mevuvik [--sizes small,lite,mid] [--batch 8] [--context 4096]
 
 ``--config 8b`` (the default) is the headline benchmark.  A step is one decode step of a batch
 of 8 sequences at a context of 8,192 tokens.  One JSON line is printed: ``value`` = decoded
@@ -118,10 +118,11 @@ def decode_bytes(model, runner, lengths, cache_bytes=None):
         per_token = g.n_layers * g.need.num_kv_heads * (g.need.head_dim + _value_dim(g)) * g.k.element_size()
         for n in lengths:
             kv += per_token * (min(n, g.need.window) if g.need.window else n)
-    # a part whose reads grow with the batch (routed experts: every expert some token chose) says so itself
+    # a part whose reads grow with the batch (routed experts: every expert some token chose) says so itself,
+    # in every run of its layer
     extra = 0
-    for block in model.blocks:
-        for part in block.parts().values():
+    for entry in model.plan.schedule:
+        for part in model.blocks[entry.layer].parts().values():
             if hasattr(part, "decode_bytes"):
                 extra += part.decode_bytes(len(lengths)) - part.weight_bytes()
     # a fixed-size state per sequence (a recurrent mixer's) is read and written once a step
@@ -293,6 +294,41 @@ def nogosun_cache_bytes(cfg, lengths, element_size=2):
     return total
 
 
+def mevuvik_prefill_flops(cfg, t):
+    """Floating-point operations of a prompt of ``t`` tokens from position 0, every run of a looped layer
+    counted: every product, the latent attention as the engine takes it (toretar_prefill_flops), scores
+    and weighted values over the causal half, the matrix memory as it is written (one update and one
+    read of the state, 4 dim vdim a head and token), the router and the chosen experts (two matrices)."""
+    import torch
+    from gemmars_b200 import kernels
+    from gemmars_b200.models.mevuvik import MevuvikConfig, runs
+    w, total, pairs = cfg["width"], 0, t * (t + 1) // 2
+    for i, _ in runs(MevuvikConfig.from_dict(cfg)):
+        m, mlp = cfg["layers"][i]["mixer"], cfg["layers"][i].get("mlp")
+        if cfg["layers"][i]["type"] == "latent_attention":
+            nh, dim, rd, vd, rq, r = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank"))
+            per_token = 2 * (w * (rq + r + rd) + rq * nh * (dim + rd) + nh * vd * w)
+            if t >= kernels.LATENT_EXPAND_MIN_TOKENS and kernels.latent_expand_usable(torch.bfloat16, r, dim, rd, vd):
+                per_token += 2 * nh * (dim + vd) * r
+                attention = 2 * nh * (dim + rd + vd) * pairs
+            else:
+                per_token += 2 * (nh * dim * r + nh * r * vd)
+                attention = 2 * nh * (2 * r + rd) * pairs
+        else:
+            a, b = m["left"], m["right"]
+            hd, hv = b["heads"] * b["dim"], b["heads"] * b["vdim"]
+            per_token = (2 * w * ((a["heads"] + a["kv_heads"]) * a["dim"] + a["kv_heads"] * a["vdim"] + a["heads"])
+                         + 2 * a["heads"] * a["vdim"] * w + 2 * w * (2 * hd + 2 * hv + 2 * b["heads"]) + 2 * hv * w
+                         + 4 * b["heads"] * b["dim"] * b["vdim"])
+            attention = 2 * a["heads"] * (a["dim"] + a["vdim"]) * pairs
+        if mlp is not None and mlp["kind"] == "dense":
+            per_token += 4 * w * mlp["ff"]
+        elif mlp is not None:
+            per_token += 2 * w * mlp["router"]["experts"] + 4 * w * mlp["router"]["top"] * mlp["expert"]["ff"]
+        total += per_token * t + attention
+    return total + 2 * w * cfg["vocab"]
+
+
 def fill_cache(runner, slots, length, real, vocab, gen):
     """Brings every slot to ``length`` cached tokens: by running prompts (real) or by
     reserving the pages and writing random keys and values (synthetic)."""
@@ -388,6 +424,8 @@ def time_prefill(eng, cfg, tokens, tflops, tflops_sustained):
         flops = dalerax_prefill_flops(cfg, tokens)
     elif cfg.get("architecture") == "Nogosun":
         flops = nogosun_prefill_flops(cfg, tokens)
+    elif cfg.get("architecture") == "Mevuvik":
+        flops = mevuvik_prefill_flops(cfg, tokens)
     elif cfg.get("sliding_window") and cfg.get("use_sliding_window"):
         size = cfg["sliding_window"]      # a window on every layer: the keys a token sees, not the causal half
         seen = sum(min(p + 1, size) for p in range(tokens))
@@ -580,10 +618,11 @@ def kernel_table(eng, tokens, batch, context):
 def run_compare(args):
     """Prompt and decode throughput of models of one architecture beside models of another with the
     same width, depth and per-token feed-forward size (Toretar and Kuporax beside Qwen3, Dalerax
-    beside Kuporax, Nogosun beside Dalerax), with a table of each one's kernels."""
-    from gemmars_b200.tuning import DALERAX_PAIRS, KUPORAX_PAIRS, NOGOSUN_PAIRS, PAIRS
-    pairs = {"kuporax": KUPORAX_PAIRS, "dalerax": DALERAX_PAIRS, "nogosun": NOGOSUN_PAIRS}.get(args.compare, PAIRS)
-    beside = {"dalerax": "kuporax", "nogosun": "dalerax"}.get(args.compare, "qwen3")
+    beside Kuporax, Nogosun beside Dalerax, Mevuvik beside Nogosun), with a table of each one's kernels."""
+    from gemmars_b200.tuning import DALERAX_PAIRS, KUPORAX_PAIRS, MEVUVIK_PAIRS, NOGOSUN_PAIRS, PAIRS
+    pairs = {"kuporax": KUPORAX_PAIRS, "dalerax": DALERAX_PAIRS, "nogosun": NOGOSUN_PAIRS,
+             "mevuvik": MEVUVIK_PAIRS}.get(args.compare, PAIRS)
+    beside = {"dalerax": "kuporax", "nogosun": "dalerax", "mevuvik": "nogosun"}.get(args.compare, "qwen3")
     hbm_gbs, tflops, tflops_sustained, peak_src = peaks()
     sizes = [s for s in args.sizes.split(",") if s]
     out = {}
@@ -622,9 +661,9 @@ def main():
     ap.add_argument("--e2e-tokens", type=int, default=E2E_TOKENS,
                     help="tokens a sequence generates in the end-to-end run (fewer for runs under a profiler)")
     ap.add_argument("--options", default="", help='further engine options, "key=value;key=value"')
-    ap.add_argument("--compare", choices=["toretar", "kuporax", "dalerax", "nogosun"], default=None,
+    ap.add_argument("--compare", choices=["toretar", "kuporax", "dalerax", "nogosun", "mevuvik"], default=None,
                     help="instead of the headline: models of that architecture beside ones of equal size (Qwen3-shaped; "
-                         "Kuporax-shaped for dalerax; Dalerax-shaped for nogosun)")
+                         "Kuporax-shaped for dalerax; Dalerax-shaped for nogosun; Nogosun-shaped for mevuvik)")
     ap.add_argument("--sizes", default="small,lite,mid", help="with --compare: which pairs of tuning.PAIRS")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -917,158 +917,330 @@ GB_EXPORT int gb_wkv_scan(const float* r, const float* k, const float* w, long l
 }
 
 // ------------------------------------------------------------------ matrix memory with exponential gates
-// The state of a head is a matrix S [dim, vdim], a vector n [dim] and a running maximum m; blocks,
-// columns, lanes and the order of S in memory as for the delta rule (dim <= 32 P).  Per token, with
-// i = cap tanh(il / cap) and f = logsigmoid(cap tanh(fl / cap)) of the gates' logits (cap 0: no cap):
+// The state of a head is a matrix S [dim, vdim], a vector n [dim] and a running maximum m.  Per token,
+// with i = cap tanh(il / cap) and f = logsigmoid(cap tanh(fl / cap)) of the gates' logits (cap 0: no cap):
 //   m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  n <- the same with k alone;
 //   y = S^T (qscale q) / (max(|n . (qscale q)|, exp(-m')) + 1e-6)
-// Tokens come in groups of GR by asynchronous copies, a group ahead.  For a group at once, before the
-// walk over its tokens: the gates (a token a thread), the running maximum (a sum and a maximum a
-// token, every lane of a warp the same, its exponentials a token a lane), and n with its products
-// n . q: thread d keeps n[d], so a token costs it two multiplications and a share of a sum that only
-// has to be there when the walk begins.  A block of 32 columns keeps an n and an m of its own
-// (aux [slots, H, blocks, 32 P + 4]: n, then m), since blocks of one head may run one after the other.
-template <int P, int GR>
-__global__ void __launch_bounds__(32 * P) matrix_memory_kernel(const float* __restrict__ q, const float* __restrict__ k,
-                                                              const float* __restrict__ v, const float* __restrict__ in_logit,
-                                                              const float* __restrict__ forget_logit, long long ld,
-                                                              float* __restrict__ state, float* __restrict__ aux,
-                                                              const int* __restrict__ cu, const int* __restrict__ seq_slot,
-                                                              float* __restrict__ y, int H, int D, int V, float cap, float qscale) {
-  constexpr int DP = P * SLICE;
-  __shared__ __align__(16) float kq[2][GR][2][padded_size(P)];   // [buffer][token][k | q][dims, padded]
-  __shared__ float vs[2][GR][32], gates[2][GR][2];
-  __shared__ float logs[GR][2], pre[GR][3];                      // i and f; then: what S keeps, what is written, exp(-m)
-  __shared__ float nq[GR][P];                                    // the warps' shares of n . q
-  pdl_wait_prior();
-  const int b = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
-  const int col = blockIdx.z * 32 + tid / P, part = tid % P, lane = tid & 31, warp = tid >> 5;
-  const bool live = col < V;
-  const int t0 = cu[b], t1 = cu[b + 1];
-  float4* Sg = (float4*)(state + ((size_t)seq_slot[b] * H + head) * 8 * V * P * 4);
-  float* ax = aux + (((size_t)seq_slot[b] * H + head) * gridDim.z + blockIdx.z) * (DP + 4);
-  float S[SLICE];
+//
+// A block is 16 columns of one (sequence, head): P lanes side by side work a column, eight dims each
+// (dim <= 8 P), and one more warp, the gate warp, does what is the same for all columns.  The walk from
+// token to token is a chain of one multiply-add an element (S <- keep S + (write v) k), so it is short
+// when a lane holds little of a column and its tokens' other work overlaps: a lane takes TB tokens'
+// read-outs before they meet over the column's lanes, in a reduction that leaves token j's sum in lane j
+// (TB - 1 shuffles for TB tokens instead of log2(P) each; with 32 dims a lane and a sum a token this
+// kernel took 0.70 us a token at dim 64).  Meanwhile the gate warp, one group of GR tokens ahead, takes
+// the gates (a gate a lane), the maxima (an addition and a maximum a token, the same in every lane), the
+// factors (a token a lane), and n with its products n . q.  Tokens come by asynchronous copies, two
+// groups ahead.  A group that ends early is walked to a multiple of TB: the tokens beyond have keep 1
+// and write 0 and change nothing.
+//
+// In memory element (d, col) of S, d = 4 P r + 4 part + e, lies at ((r * vdim + col) * P + part) * 4 + e
+// (8 P vdim floats a head).  A block keeps an n and an m of its own (aux [slots, H, blocks, 8 P + 4]: n,
+// then m), since blocks of one head may run one after the other.
+constexpr int MM_COLS = 16;
+template <int P, int TB>
+__device__ __forceinline__ float tokens_sum(float (&a)[TB], int part) {   // the column's sum for token part % TB
 #pragma unroll
-  for (int r = 0; r < SLICE / 4; ++r) {
-    const float4 s4 = live ? Sg[((size_t)r * V + col) * P + part] : make_float4(0.f, 0.f, 0.f, 0.f);
-    S[4 * r] = s4.x; S[4 * r + 1] = s4.y; S[4 * r + 2] = s4.z; S[4 * r + 3] = s4.w;
+  for (int o = P / 2; o >= TB; o >>= 1)
+#pragma unroll
+    for (int j = 0; j < TB; ++j) a[j] += __shfl_xor_sync(0xffffffffu, a[j], o);
+#pragma unroll
+  for (int o = (TB < P ? TB : P) / 2; o >= 1; o >>= 1) {
+    const bool upper = (part & o) != 0;
+#pragma unroll
+    for (int j = 0; j < o; ++j) {
+      const float give = upper ? a[j] : a[j + o], kept = upper ? a[j + o] : a[j];
+      a[j] = kept + __shfl_xor_sync(0xffffffffu, give, o);
+    }
   }
-  float nd = ax[tid], m = ax[DP];
-  if (tid >= D)      // the dims beyond the head's are zeros, written once
-    for (int j = 0; j < 2 * GR; ++j) kq[j / GR][j % GR][0][padded(tid)] = kq[j / GR][j % GR][1][padded(tid)] = 0.f;
-  auto bring = [&](int first, int buf) {
-    for (int j = 0; j < GR && first + j < t1; ++j) {
-      const size_t t = first + j;
-      if (tid < D) {
-        copy_async4(&kq[buf][j][0][padded(tid)], k + t * ld + head * D + tid);
-        copy_async4(&kq[buf][j][1][padded(tid)], q + t * ld + head * D + tid);
+  return a[0];
+}
+__device__ __forceinline__ void copy_async16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+template <int P, int GR, int TB>
+__global__ void __launch_bounds__(MM_COLS * P + 32) matrix_memory_kernel(const float* __restrict__ q, const float* __restrict__ k,
+                                                                        const float* __restrict__ v, const float* __restrict__ in_logit,
+                                                                        const float* __restrict__ forget_logit, long long ld,
+                                                                        float* __restrict__ state, float* __restrict__ aux,
+                                                                        const int* __restrict__ cu, const int* __restrict__ seq_slot,
+                                                                        float* __restrict__ y, int H, int D, int V, float cap,
+                                                                        float qscale, int wide) {
+  static_assert(TB <= P && GR % TB == 0 && 2 * GR <= 32, "a lane for every token of a batch, a lane for every gate of a group");
+  constexpr int DP = 8 * P, WALKERS = MM_COLS * P, NL = DP / 32;
+  __shared__ __align__(16) float kq[3][GR][2][DP];   // [buffer][token][k | q]
+  __shared__ __align__(16) float vs[3][GR][MM_COLS];
+  __shared__ float pre[2][GR][3];                    // what S keeps, what is written, the factor on the read-out
+  pdl_wait_prior();
+  const int b = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, col0 = blockIdx.z * MM_COLS;
+  const int t0 = cu[b], t1 = cu[b + 1], groups = (t1 - t0 + GR - 1) / GR;
+  const bool gates = tid >= WALKERS;
+  const int lane = tid & 31, part = tid % P, mine = tid / P, col = col0 + mine;
+  const bool live = !gates && col < V;
+  float4* Sg = (float4*)(state + ((size_t)seq_slot[b] * H + head) * 2 * V * P * 4);
+  float* ax = aux + (((size_t)seq_slot[b] * H + head) * gridDim.z + blockIdx.z) * (DP + 4);
+  {   // dims beyond the head's, columns beyond the last and tokens beyond the end are zeros
+    const int used = min(3, groups) * GR;
+    for (int i = tid; i < used * 2 * DP / 4; i += WALKERS + 32) ((float4*)kq)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = tid; i < used * MM_COLS; i += WALKERS + 32) ((float*)vs)[i] = 0.f;
+  }
+  __syncthreads();
+  // the walkers bring a group's rows of k, q and v; `wide`: they can be read sixteen bytes at a time
+  auto bring = [&](int group) {
+    const int first = t0 + group * GR, n = min(GR, t1 - first), buf = group % 3;
+    const int cols = min(MM_COLS, V - col0);
+    if (wide) {
+      const int per = D / 4, vper = cols / 4;
+      for (int i = tid; i < n * 2 * per; i += WALKERS) {
+        const int j = i / (2 * per), c = i % (2 * per), which = c / per, d = (c % per) * 4;
+        copy_async16(&kq[buf][j][which][d], (which ? q : k) + (size_t)(first + j) * ld + head * D + d);
       }
-      if (live && part == 0) copy_async4(&vs[buf][j][tid / P], v + t * ld + head * V + col);
-      if (tid == 0) copy_async4(&gates[buf][j][0], in_logit + t * ld + head);
-      if (tid == 1) copy_async4(&gates[buf][j][1], forget_logit + t * ld + head);
+      for (int i = tid; i < n * vper; i += WALKERS) {
+        const int j = i / vper, c = (i % vper) * 4;
+        copy_async16(&vs[buf][j][c], v + (size_t)(first + j) * ld + head * V + col0 + c);
+      }
+    } else {
+      for (int i = tid; i < n * 2 * D; i += WALKERS) {
+        const int j = i / (2 * D), c = i % (2 * D), which = c / D, d = c % D;
+        copy_async4(&kq[buf][j][which][d], (which ? q : k) + (size_t)(first + j) * ld + head * D + d);
+      }
+      for (int i = tid; i < n * cols; i += WALKERS) {
+        const int j = i / cols, c = i % cols;
+        copy_async4(&vs[buf][j][c], v + (size_t)(first + j) * ld + head * V + col0 + c);
+      }
     }
     copy_async_commit();
   };
-  bring(t0, 0);
-  for (int first = t0; first < t1; first += GR) {
-    const int buf = ((first - t0) / GR) & 1;
-    if (first + GR < t1) {
-      bring(first + GR, buf ^ 1);
-      copy_async_wait<1>();
-    } else {
-      copy_async_wait<0>();
-    }
-    __syncthreads();
-    const int n = min(GR, t1 - first);
-    if (tid < 2 * n) {                        // a gate a thread: 2 GR <= 32, so one warp has them all
-      const int j = tid >> 1;
-      float z = gates[buf][j][tid & 1];
-      if (cap > 0.f) z = cap * tanhf(z / cap);
-      logs[j][tid & 1] = (tid & 1) ? -softplus_f(-z) : z;
-    }
-    __syncthreads();
-    {                                         // every warp takes the maxima for itself; warp 0 leaves the factors
-      float before = m, mine_before = 0.f, mine = 0.f;
-      for (int j = 0; j < n; ++j) {
-        const float now = fmaxf(logs[j][1] + before, logs[j][0]);
-        if (lane == j) { mine_before = before; mine = now; }
-        before = now;
-      }
-      m = before;
-      float keep = 0.f, write = 0.f;
-      if (lane < n) {
-        keep = expf(logs[lane][1] + mine_before - mine);
-        write = expf(logs[lane][0] - mine);
-        if (warp == 0) {
-          pre[lane][0] = keep;
-          pre[lane][1] = write;
-          pre[lane][2] = expf(-mine);
-        }
-      }
-      for (int j = 0; j < n; ++j) {
-        const float kp = __shfl_sync(0xffffffffu, keep, j), wr = __shfl_sync(0xffffffffu, write, j);
-        nd = fmaf(wr, kq[buf][j][0][padded(tid)], kp * nd);
-        const float s = warp_sum(nd * kq[buf][j][1][padded(tid)]);
-        if (lane == 0) nq[j][warp] = s;
-      }
-    }
-    __syncthreads();
-    for (int j = 0; j < n; ++j) {
-      const float4* ks = (const float4*)(kq[buf][j][0] + part * (SLICE + 4));
-      const float4* qs = (const float4*)(kq[buf][j][1] + part * (SLICE + 4));
-      const float keep = pre[j][0], wv = pre[j][1] * (live ? vs[buf][j][tid / P] : 0.f);
-      float acc = 0.f, acc2 = 0.f;
+  // ---- the gate warp's part of a group
+  float nd[NL], m = 0.f, raw = 0.f;
+  auto fetch_logit = [&](int group) {                // lane j: the input gate of token j; lane GR + j: its forget gate
+    const int t = t0 + group * GR + lane % GR;
+    raw = (lane < 2 * GR && t < t1) ? (lane < GR ? in_logit : forget_logit)[(size_t)t * ld + head] : 0.f;
+  };
+  auto take_gates = [&](int group) {
+    const int n = min(GR, t1 - (t0 + group * GR)), buf = group % 3;
+    float z = cap > 0.f ? cap * tanhf(raw / cap) : raw;
+    if (lane >= GR) z = -softplus_f(-z);
+    if (group + 1 < groups) fetch_logit(group + 1);
+    float before = m, from = 0.f, to = 0.f;
 #pragma unroll
-      for (int r = 0; r < SLICE / 4; ++r) {
-        const float4 kv = ks[r], qv = qs[r];
-        S[4 * r] = fmaf(kv.x, wv, keep * S[4 * r]);         acc = fmaf(S[4 * r], qv.x, acc);
-        S[4 * r + 1] = fmaf(kv.y, wv, keep * S[4 * r + 1]); acc2 = fmaf(S[4 * r + 1], qv.y, acc2);
-        S[4 * r + 2] = fmaf(kv.z, wv, keep * S[4 * r + 2]); acc = fmaf(S[4 * r + 2], qv.z, acc);
-        S[4 * r + 3] = fmaf(kv.w, wv, keep * S[4 * r + 3]); acc2 = fmaf(S[4 * r + 3], qv.w, acc2);
-      }
-      acc = lanes_sum<P>(acc + acc2);
-      if (live && part == 0) {
-        float dot = nq[j][0];
+    for (int j = 0; j < GR; ++j) {
+      const float i = __shfl_sync(0xffffffffu, z, j), f = __shfl_sync(0xffffffffu, z, GR + j);
+      const float now = j < n ? fmaxf(f + before, i) : before;
+      if (lane == j) { from = before; to = now; }
+      before = now;
+    }
+    m = before;
+    const float f = __shfl_sync(0xffffffffu, z, GR + lane % GR);
+    const float keep = lane < n ? expf(f + from - to) : 1.f, write = lane < n ? expf(z - to) : 0.f;
+    float dots[GR];
 #pragma unroll
-        for (int w = 1; w < P; ++w) dot += nq[j][w];
-        y[(size_t)(first + j) * H * V + head * V + col] = acc * qscale / (fmaxf(fabsf(dot * qscale), pre[j][2]) + 1e-6f);
+    for (int j = 0; j < GR; ++j) {
+      const float kp = __shfl_sync(0xffffffffu, keep, j), wr = __shfl_sync(0xffffffffu, write, j);
+      dots[j] = 0.f;
+#pragma unroll
+      for (int u = 0; u < NL; ++u) {
+        nd[u] = fmaf(kp, nd[u], wr * kq[buf][j][0][lane + 32 * u]);
+        dots[j] = fmaf(nd[u], kq[buf][j][1][lane + 32 * u], dots[j]);
       }
     }
-    __syncthreads();   // the group after next is brought into this buffer; pre and nq are written again
+    const float dot = tokens_sum<32, GR>(dots, lane);     // lane j: token j's
+    if (lane < GR) {
+      pre[group & 1][lane][0] = keep;
+      pre[group & 1][lane][1] = write;
+      pre[group & 1][lane][2] = qscale / (fmaxf(fabsf(dot * qscale), expf(-to)) + 1e-6f);
+    }
+  };
+  float S[8];
+  if (gates) {
+#pragma unroll
+    for (int u = 0; u < NL; ++u) nd[u] = ax[lane + 32 * u];
+    m = ax[DP];
+    fetch_logit(0);
+  } else {
+    bring(0);
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const float4 s4 = live ? Sg[((size_t)r * V + col) * P + part] : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[4 * r] = s4.x; S[4 * r + 1] = s4.y; S[4 * r + 2] = s4.z; S[4 * r + 3] = s4.w;
+    }
+    copy_async_wait<0>();
+  }
+  __syncthreads();
+  if (gates) {
+    if (groups > 0) take_gates(0);
+  } else if (groups > 1) {
+    bring(1);
+  }
+  for (int g = 0; g < groups; ++g) {
+    copy_async_wait<0>();
+    __syncthreads();         // group g + 1 has arrived, the gates of group g are taken, everyone has left group g - 1
+    if (gates) {
+      if (g + 1 < groups) take_gates(g + 1);
+      continue;
+    }
+    if (g + 2 < groups) bring(g + 2);
+    const int buf = g % 3, first = t0 + g * GR, n = min(GR, t1 - first);
+#pragma unroll 1
+    for (int j0 = 0; j0 < n; j0 += TB) {
+      float acc[TB];
+#pragma unroll
+      for (int j = 0; j < TB; ++j) {
+        const float keep = pre[g & 1][j0 + j][0], wv = pre[g & 1][j0 + j][1] * vs[buf][j0 + j][mine];
+        const float4 k0 = *(const float4*)&kq[buf][j0 + j][0][4 * part], k1 = *(const float4*)&kq[buf][j0 + j][0][4 * (P + part)];
+        const float4 q0 = *(const float4*)&kq[buf][j0 + j][1][4 * part], q1 = *(const float4*)&kq[buf][j0 + j][1][4 * (P + part)];
+        S[0] = fmaf(keep, S[0], wv * k0.x); S[1] = fmaf(keep, S[1], wv * k0.y);
+        S[2] = fmaf(keep, S[2], wv * k0.z); S[3] = fmaf(keep, S[3], wv * k0.w);
+        S[4] = fmaf(keep, S[4], wv * k1.x); S[5] = fmaf(keep, S[5], wv * k1.y);
+        S[6] = fmaf(keep, S[6], wv * k1.z); S[7] = fmaf(keep, S[7], wv * k1.w);
+        float a = S[0] * q0.x, c = S[4] * q1.x;
+        a = fmaf(S[1], q0.y, a); c = fmaf(S[5], q1.y, c);
+        a = fmaf(S[2], q0.z, a); c = fmaf(S[6], q1.z, c);
+        a = fmaf(S[3], q0.w, a); c = fmaf(S[7], q1.w, c);
+        acc[j] = a + c;
+      }
+      const float sum = tokens_sum<P, TB>(acc, part);
+      const int j = j0 + part % TB;
+      if (live && part < TB && j < n) y[(size_t)(first + j) * H * V + head * V + col] = sum * pre[g & 1][j][2];
+    }
   }
   // only now may the kernel after this one start: its waiting blocks would take the room of this
-  // kernel's few warps, which are a chain from token to token
+  // kernel's warps, which are a chain from token to token
   pdl_release_next();
-  ax[tid] = nd;
-  if (tid == 0) ax[DP] = m;
-  if (live) {
+  if (gates) {
 #pragma unroll
-    for (int r = 0; r < SLICE / 4; ++r)
-      Sg[((size_t)r * V + col) * P + part] = make_float4(S[4 * r], S[4 * r + 1], S[4 * r + 2], S[4 * r + 3]);
+    for (int u = 0; u < NL; ++u) ax[lane + 32 * u] = nd[u];
+    if (lane == 0) ax[DP] = m;
+  } else if (live) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) Sg[((size_t)r * V + col) * P + part] = make_float4(S[4 * r], S[4 * r + 1], S[4 * r + 2], S[4 * r + 3]);
   }
 }
 
-// Floats of one head's n and m (what a caller allocates per slot and head): one set per 32 columns.
-GB_EXPORT int gb_matrix_memory_aux_floats(int dims, int V) { return (V + 31) / 32 * (lanes_for(dims) * SLICE + 4); }
+// A step of single tokens: a warp is 16 columns of one (sequence, head) with their own n and m, and needs
+// nothing of the others.  It asks for its share of the state, then takes the gates and n . q (every lane
+// the scalars, NL dims of n each) while that is on its way.
+template <int P>
+__global__ void __launch_bounds__(128) matrix_memory_single_kernel(const float* __restrict__ q, const float* __restrict__ k,
+                                                                  const float* __restrict__ v, const float* __restrict__ in_logit,
+                                                                  const float* __restrict__ forget_logit, long long ld,
+                                                                  float* __restrict__ state, float* __restrict__ aux,
+                                                                  const int* __restrict__ seq_slot, float* __restrict__ y, int units,
+                                                                  int blocks, int H, int D, int V, float cap, float qscale) {
+  constexpr int DP = 8 * P, NL = DP / 32, WC = 32 / P, ITER = MM_COLS / WC, AT = ITER < 4 ? ITER : 4;
+  pdl_release_next();
+  pdl_wait_prior();
+  const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, part = lane % P;
+  if (unit >= units) return;
+  const int z = unit % blocks, head = unit / blocks % H, t = unit / blocks / H, col0 = z * MM_COLS;
+  const size_t hs = (size_t)seq_slot[t] * H + head;
+  float4* Sg = (float4*)(state + hs * 2 * V * P * 4);
+  float* ax = aux + (hs * blocks + z) * (DP + 4);
+  const float* krow = k + (size_t)t * ld + head * D;
+  const float* qrow = q + (size_t)t * ld + head * D;
+  float4 s0[AT], s1[AT];
+  auto load = [&](int it) {
+#pragma unroll
+    for (int u = 0; u < AT; ++u) {
+      const int col = col0 + (it + u) * WC + lane / P;
+      const bool live = col < V;
+      s0[u] = live ? Sg[(size_t)col * P + part] : make_float4(0.f, 0.f, 0.f, 0.f);
+      s1[u] = live ? Sg[((size_t)V + col) * P + part] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  load(0);
+  float kd[8], qd[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    const int d = (e >> 2) * 4 * P + 4 * part + (e & 3);
+    kd[e] = d < D ? krow[d] : 0.f;
+    qd[e] = d < D ? qrow[d] : 0.f;
+  }
+  float zi = in_logit[(size_t)t * ld + head], zf = forget_logit[(size_t)t * ld + head];
+  if (cap > 0.f) {
+    zi = cap * tanhf(zi / cap);
+    zf = cap * tanhf(zf / cap);
+  }
+  zf = -softplus_f(-zf);
+  const float m = ax[DP], now = fmaxf(zf + m, zi), keep = expf(zf + m - now), write = expf(zi - now);
+  float dot = 0.f;
+#pragma unroll
+  for (int u = 0; u < NL; ++u) {
+    const int d = lane + 32 * u;
+    const float nd = fmaf(keep, ax[d], write * (d < D ? krow[d] : 0.f));
+    dot = fmaf(nd, d < D ? qrow[d] : 0.f, dot);
+    ax[d] = nd;
+  }
+  dot = warp_sum(dot);       // every lane has read m by now
+  if (lane == 0) ax[DP] = now;
+  const float factor = qscale / (fmaxf(fabsf(dot * qscale), expf(-now)) + 1e-6f);
+#pragma unroll 1
+  for (int it = 0; it < ITER; it += AT) {
+    if (it > 0) load(it);
+#pragma unroll
+    for (int u = 0; u < AT; ++u) {
+      const int col = col0 + (it + u) * WC + lane / P;
+      const bool live = col < V;
+      const float wv = live ? write * v[(size_t)t * ld + head * V + col] : 0.f;
+      float4 a = s0[u], c = s1[u];
+      a.x = fmaf(keep, a.x, wv * kd[0]); a.y = fmaf(keep, a.y, wv * kd[1]); a.z = fmaf(keep, a.z, wv * kd[2]); a.w = fmaf(keep, a.w, wv * kd[3]);
+      c.x = fmaf(keep, c.x, wv * kd[4]); c.y = fmaf(keep, c.y, wv * kd[5]); c.z = fmaf(keep, c.z, wv * kd[6]); c.w = fmaf(keep, c.w, wv * kd[7]);
+      if (live) {
+        Sg[(size_t)col * P + part] = a;
+        Sg[((size_t)V + col) * P + part] = c;
+      }
+      float r0 = a.x * qd[0], r1 = c.x * qd[4];
+      r0 = fmaf(a.y, qd[1], r0); r1 = fmaf(c.y, qd[5], r1);
+      r0 = fmaf(a.z, qd[2], r0); r1 = fmaf(c.z, qd[6], r1);
+      r0 = fmaf(a.w, qd[3], r0); r1 = fmaf(c.w, qd[7], r1);
+      const float sum = lanes_sum<P>(r0 + r1);
+      if (live && part == 0) y[(size_t)t * H * V + head * V + col] = sum * factor;
+    }
+  }
+}
+
+static inline int mm_lanes(int dims) { return dims <= 32 ? 4 : (dims <= 64 ? 8 : (dims <= 128 ? 16 : 32)); }
+
+// Floats of one head's S, and of its n and m (what a caller allocates per slot and head).
+GB_EXPORT int gb_matrix_memory_floats(int dims, int V) { return 8 * mm_lanes(dims) * V; }
+GB_EXPORT int gb_matrix_memory_aux_floats(int dims, int V) { return (V + MM_COLS - 1) / MM_COLS * (8 * mm_lanes(dims) + 4); }
 
 // q, k: rows of ld floats, head h at h * D; v: head h at h * V; in_logit, forget_logit: [ntok, H] in rows of ld;
-// state: [slots, H, gb_state_floats(D, V)], aux: [slots, H, gb_matrix_memory_aux_floats(D, V)] float32, zeros
-// for a new sequence; y: [ntok, H * V].  cap: the gates' cap (0: none).
+// state: [slots, H, gb_matrix_memory_floats(D, V)], aux: [slots, H, gb_matrix_memory_aux_floats(D, V)] float32,
+// zeros for a new sequence; y: [ntok, H * V].  cap: the gates' cap (0: none).  ntok == nseq: every sequence
+// brings one token.
 GB_EXPORT int gb_matrix_memory(const float* q, const float* k, const float* v, const float* in_logit, const float* forget_logit,
-                               long long ld, float* state, float* aux, const int* cu, const int* seq_slot, float* y, int nseq,
+                               long long ld, float* state, float* aux, const int* cu, const int* seq_slot, float* y, int ntok, int nseq,
                                int H, int D, int V, float cap, float qscale, cudaStream_t stream) {
   if (nseq <= 0) return 0;
-  if (H <= 0 || V <= 0 || D <= 0 || D > 8 * SLICE || ((uintptr_t)state & 15)) return GB_ERR_SIZE;
+  if (H <= 0 || V <= 0 || D <= 0 || D > 256 || ((uintptr_t)state & 15)) return GB_ERR_SIZE;
   if (cap < 0.f) return GB_ERR_ARG;
-  dim3 grid(nseq, H, (V + 31) / 32);
-#define GB_MEMORY(P, GR)                                                                                                \
-  launch_scan(matrix_memory_kernel<P, GR>, grid, 32 * P, stream, q, k, v, in_logit, forget_logit, ld, state, aux, cu, seq_slot, y, \
-              H, D, V, cap, qscale)
-  switch (lanes_for(D)) {
-    case 1: GB_MEMORY(1, 8); break;
-    case 2: GB_MEMORY(2, 8); break;
-    case 4: GB_MEMORY(4, 8); break;
-    default: GB_MEMORY(8, 8);
+  const int wide = D % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && !(((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 15);
+  dim3 grid(nseq, H, (V + MM_COLS - 1) / MM_COLS);
+  if (ntok == nseq) {                          // every sequence brings one token
+    const long long units = (long long)nseq * H * grid.z;
+    if (units > 0x7fffffff) return GB_ERR_SIZE;
+#define GB_MEMORY(P)                                                                                                          \
+  gb_launch(matrix_memory_single_kernel<P>, dim3((unsigned)((units + 3) / 4)), 128, 0, stream, q, k, v, in_logit, forget_logit, \
+            ld, state, aux, seq_slot, y, (int)units, (int)grid.z, H, D, V, cap, qscale)
+    switch (mm_lanes(D)) {
+      case 4: GB_MEMORY(4); break;
+      case 8: GB_MEMORY(8); break;
+      case 16: GB_MEMORY(16); break;
+      default: GB_MEMORY(32);
+    }
+#undef GB_MEMORY
+    return gb_launch_status();
+  }
+#define GB_MEMORY(P, GR, TB)                                                                                                  \
+  launch_scan(matrix_memory_kernel<P, GR, TB>, grid, MM_COLS * P + 32, stream, q, k, v, in_logit, forget_logit, ld, state, aux, \
+              cu, seq_slot, y, H, D, V, cap, qscale, wide)
+  switch (mm_lanes(D)) {
+    case 4: GB_MEMORY(4, 16, 4); break;
+    case 8: GB_MEMORY(8, 16, 8); break;
+    case 16: GB_MEMORY(16, 8, 8); break;
+    default: GB_MEMORY(32, 4, 4);
   }
 #undef GB_MEMORY
   return gb_launch_status();

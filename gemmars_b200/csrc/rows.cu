@@ -181,25 +181,33 @@ GB_EXPORT int gb_cap_f32(float* y, long long total, float cap, cudaStream_t stre
   return gb_launch_status();
 }
 
-// One block a row: in(i) gives the row's element i, out(i, normed) takes it.  The row is kept in
-// registers between the passes where it fits, else read again; the order of the additions depends on
-// n and the block size alone.
-template <typename In, typename Out>
+// One block a row.  V elements at a time (4 where rows and their starts allow sixteen-byte accesses, else
+// 1): in(i, v) reads the row's elements V i .. V i + V - 1, out(i, v, inv) takes them again with the factor
+// that norms them.  The row is kept in registers between the passes where it fits, else read again; the
+// order of the additions depends on n, V and the block size alone.
+template <int V, typename In, typename Out>
 __device__ __forceinline__ void norm_row(int n, float eps, float* scratch, In in, Out out) {
-  constexpr int KEEP = 8;
-  float held[KEEP], ss = 0.f;
-  const bool keep = n <= KEEP * (int)blockDim.x;
+  constexpr int KEEP = V == 4 ? 4 : 8;
+  const int pieces = n / V;
+  float held[KEEP][V], ss = 0.f;
+  const bool keep = pieces <= KEEP * (int)blockDim.x;
   if (keep) {
 #pragma unroll
     for (int u = 0; u < KEEP; ++u) {
       const int i = threadIdx.x + u * blockDim.x;
-      held[u] = i < n ? in(i) : 0.f;
-      ss = fmaf(held[u], held[u], ss);
+      if (i < pieces) in(i, held[u]);
     }
+#pragma unroll
+    for (int u = 0; u < KEEP; ++u)
+      if (threadIdx.x + u * blockDim.x < pieces)
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss = fmaf(held[u][e], held[u][e], ss);
   } else {
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-      const float v = in(i);
-      ss = fmaf(v, v, ss);
+    for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+      float v[V];
+      in(i, v);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
     }
   }
   const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
@@ -207,17 +215,41 @@ __device__ __forceinline__ void norm_row(int n, float eps, float* scratch, In in
 #pragma unroll
     for (int u = 0; u < KEEP; ++u) {
       const int i = threadIdx.x + u * blockDim.x;
-      if (i < n) out(i, held[u] * inv);
+      if (i < pieces) out(i, held[u], inv);
     }
   } else {
-    for (int i = threadIdx.x; i < n; i += blockDim.x) out(i, in(i) * inv);
+    for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+      float v[V];
+      in(i, v);
+      out(i, v, inv);
+    }
   }
 }
-static inline int row_threads(int n) { return n >= 2048 ? 512 : (n >= 512 ? 256 : 128); }
+static inline int row_threads(int n) { return n >= 2048 ? 256 : 128; }
+
+// Elements V i .. V i + V - 1 of a row, V of them in one access.
+__device__ __forceinline__ void take(const float* p, int i, float (&v)[1]) { v[0] = p[i]; }
+__device__ __forceinline__ void take(const bf16* p, int i, float (&v)[1]) { v[0] = to_f32(p[i]); }
+__device__ __forceinline__ void take(const float* p, int i, float (&v)[4]) {
+  const float4 a = ((const float4*)p)[i];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void take(const bf16* p, int i, float (&v)[4]) {
+  const uint2 a = ((const uint2*)p)[i];
+  const float2 lo = __bfloat1622float2(*(const __nv_bfloat162*)&a.x), hi = __bfloat1622float2(*(const __nv_bfloat162*)&a.y);
+  v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+}
+template <typename O> __device__ __forceinline__ void give(O* p, int i, const float (&v)[1]) { p[i] = from_f32<O>(v[0]); }
+__device__ __forceinline__ void give(float* p, int i, const float (&v)[4]) { ((float4*)p)[i] = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void give(bf16* p, int i, const float (&v)[4]) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+  ((uint2*)p)[i] = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+}
+static inline bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
 // x[t, :] = rmsnorm(table[tokens[t], :] * scale) * w
-template <typename W>
-__global__ void __launch_bounds__(512) embed_norm_kernel(const W* __restrict__ table, const int* __restrict__ tokens,
+template <typename W, int V>
+__global__ void __launch_bounds__(256) embed_norm_kernel(const W* __restrict__ table, const int* __restrict__ tokens,
                                                          const float* __restrict__ w, float* __restrict__ x, int hidden, int rows,
                                                          float scale, float eps) {
   __shared__ float scratch[33];
@@ -226,8 +258,20 @@ __global__ void __launch_bounds__(512) embed_norm_kernel(const W* __restrict__ t
   int id = tokens[blockIdx.x];
   id = id < 0 ? 0 : (id >= rows ? rows - 1 : id);
   const W* row = table + (size_t)id * hidden;
-  float* out = x + (size_t)blockIdx.x * hidden;
-  norm_row(hidden, eps, scratch, [&](int i) { return to_f32(row[i]) * scale; }, [&](int i, float v) { out[i] = v * w[i]; });
+  float* o = x + (size_t)blockIdx.x * hidden;
+  norm_row<V>(hidden, eps, scratch,
+              [&](int i, float (&v)[V]) {
+                take(row, i, v);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] *= scale;
+              },
+              [&](int i, float (&v)[V], float inv) {
+                float g[V];
+                take(w, i, g);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] = v[e] * inv * g[e];
+                give(o, i, v);
+              });
 }
 
 GB_EXPORT int gb_embed_norm(const void* table, int table_dtype, const int* tokens, const float* w, float* x, int ntok, int hidden,
@@ -235,18 +279,18 @@ GB_EXPORT int gb_embed_norm(const void* table, int table_dtype, const int* token
   if (ntok <= 0) return 0;
   if (hidden <= 0 || rows <= 0) return GB_ERR_SIZE;
   const int threads = row_threads(hidden);
-  if (table_dtype == GB_F32)
-    gb_launch(embed_norm_kernel<float>, ntok, threads, 0, stream, (const float*)table, tokens, w, x, hidden, rows, scale, eps);
-  else if (table_dtype == GB_BF16)
-    gb_launch(embed_norm_kernel<bf16>, ntok, threads, 0, stream, (const bf16*)table, tokens, w, x, hidden, rows, scale, eps);
-  else
-    return GB_ERR_DTYPE;
+  const bool four = hidden % 4 == 0 && aligned16(table) && aligned16(w) && aligned16(x);
+#define LAUNCH(W, V) gb_launch(embed_norm_kernel<W, V>, ntok, threads, 0, stream, (const W*)table, tokens, w, x, hidden, rows, scale, eps)
+  if (table_dtype == GB_F32) { if (four) LAUNCH(float, 4); else LAUNCH(float, 1); }
+  else if (table_dtype == GB_BF16) { if (four) LAUNCH(bf16, 4); else LAUNCH(bf16, 1); }
+  else return GB_ERR_DTYPE;
+#undef LAUNCH
   return gb_launch_status();
 }
 
 // x[t, :] += v for every row, and, when a weight is given, h[t, :] = rmsnorm(x[t, :]) * w of the new rows
-template <typename O>
-__global__ void __launch_bounds__(512) add_row_norm_kernel(const float* __restrict__ v, float* __restrict__ x, int n,
+template <typename O, int V>
+__global__ void __launch_bounds__(256) add_row_norm_kernel(const float* __restrict__ v, float* __restrict__ x, int n,
                                                            const float* __restrict__ w, O* __restrict__ h, float eps) {
   __shared__ float scratch[33];
   pdl_release_next();
@@ -257,12 +301,23 @@ __global__ void __launch_bounds__(512) add_row_norm_kernel(const float* __restri
     return;
   }
   O* hrow = h + (size_t)blockIdx.x * n;
-  // a thread reads, in both passes of a long row, only elements that it wrote or that nobody has written yet
-  norm_row(n, eps, scratch, [&](int i) { return row[i] + v[i]; },
-           [&](int i, float normed) {
-             hrow[i] = from_f32<O>(normed * w[i]);
-             row[i] += v[i];
-           });
+  // a thread reads, in both passes of a long row, only elements that nobody else writes
+  norm_row<V>(n, eps, scratch,
+              [&](int i, float (&r)[V]) {
+                float add[V];
+                take(row, i, r);
+                take(v, i, add);
+#pragma unroll
+                for (int e = 0; e < V; ++e) r[e] += add[e];
+              },
+              [&](int i, float (&r)[V], float inv) {
+                float g[V];
+                take(w, i, g);
+                give(row, i, r);
+#pragma unroll
+                for (int e = 0; e < V; ++e) r[e] = r[e] * inv * g[e];
+                give(hrow, i, r);
+              });
 }
 
 GB_EXPORT int gb_add_row_norm(const float* v, float* x, int rows, int n, const float* w, void* h, int h_dtype, float eps,
@@ -270,25 +325,32 @@ GB_EXPORT int gb_add_row_norm(const float* v, float* x, int rows, int n, const f
   if (rows <= 0) return 0;
   if (n <= 0) return GB_ERR_SIZE;
   const int threads = row_threads(n);
-  if (w && h_dtype == GB_BF16)
-    gb_launch(add_row_norm_kernel<bf16>, rows, threads, 0, stream, v, x, n, w, (bf16*)h, eps);
-  else if (!w || h_dtype == GB_F32)
-    gb_launch(add_row_norm_kernel<float>, rows, threads, 0, stream, v, x, n, w, (float*)h, eps);
-  else
-    return GB_ERR_DTYPE;
+  const bool four = n % 4 == 0 && aligned16(v) && aligned16(x) && aligned16(w) && aligned16(h);
+#define LAUNCH(O, V) gb_launch(add_row_norm_kernel<O, V>, rows, threads, 0, stream, v, x, n, w, (O*)h, eps)
+  if (w && h_dtype == GB_BF16) { if (four) LAUNCH(bf16, 4); else LAUNCH(bf16, 1); }
+  else if (!w || h_dtype == GB_F32) { if (four) LAUNCH(float, 4); else LAUNCH(float, 1); }
+  else return GB_ERR_DTYPE;
+#undef LAUNCH
   return gb_launch_status();
 }
 
 // out[t, :] = rmsnorm(x[t, :n]) * w for rows of x that are ldx floats apart
-template <typename O>
-__global__ void __launch_bounds__(512) norm_cols_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w,
+template <typename O, int V>
+__global__ void __launch_bounds__(256) norm_cols_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w,
                                                         O* __restrict__ out, int n, float eps) {
   __shared__ float scratch[33];
   pdl_release_next();
   pdl_wait_prior();
   const float* row = x + (size_t)blockIdx.x * ldx;
   O* o = out + (size_t)blockIdx.x * n;
-  norm_row(n, eps, scratch, [&](int i) { return row[i]; }, [&](int i, float v) { o[i] = from_f32<O>(v * w[i]); });
+  norm_row<V>(n, eps, scratch, [&](int i, float (&v)[V]) { take(row, i, v); },
+              [&](int i, float (&v)[V], float inv) {
+                float g[V];
+                take(w, i, g);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] = v[e] * inv * g[e];
+                give(o, i, v);
+              });
 }
 
 GB_EXPORT int gb_norm_cols(const float* x, long long ldx, const float* w, void* out, int out_dtype, int rows, int n, float eps,
@@ -296,11 +358,11 @@ GB_EXPORT int gb_norm_cols(const float* x, long long ldx, const float* w, void* 
   if (rows <= 0) return 0;
   if (n <= 0) return GB_ERR_SIZE;
   const int threads = row_threads(n);
-  if (out_dtype == GB_F32)
-    gb_launch(norm_cols_kernel<float>, rows, threads, 0, stream, x, ldx, w, (float*)out, n, eps);
-  else if (out_dtype == GB_BF16)
-    gb_launch(norm_cols_kernel<bf16>, rows, threads, 0, stream, x, ldx, w, (bf16*)out, n, eps);
-  else
-    return GB_ERR_DTYPE;
+  const bool four = n % 4 == 0 && ldx % 4 == 0 && aligned16(x) && aligned16(w) && aligned16(out);
+#define LAUNCH(O, V) gb_launch(norm_cols_kernel<O, V>, rows, threads, 0, stream, x, ldx, w, (O*)out, n, eps)
+  if (out_dtype == GB_F32) { if (four) LAUNCH(float, 4); else LAUNCH(float, 1); }
+  else if (out_dtype == GB_BF16) { if (four) LAUNCH(bf16, 4); else LAUNCH(bf16, 1); }
+  else return GB_ERR_DTYPE;
+#undef LAUNCH
   return gb_launch_status();
 }

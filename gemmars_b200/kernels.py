@@ -1819,11 +1819,23 @@ def wkv_scan(r, k, w, v, bonus, state, cu_seqlens, seq_slot, y, heads, dim, vdim
            _nbytes(y) * 5 + 2 * seq_slot.numel() * heads * dim * vdim * 4)
 
 
+def matrix_memory_floats(dims: int, vdim: int) -> int:
+    """Floats per head that ``matrix_memory`` keeps for its state matrix [dims, vdim]: the dims padded to
+    32, 64, 128 or 256, in the order the kernel's lanes read them (see matrix_memory_matrix)."""
+    return (32 if dims <= 32 else (64 if dims <= 64 else (128 if dims <= 128 else 256))) * vdim
+
+
+def matrix_memory_matrix(head_state: torch.Tensor, dims: int, vdim: int) -> torch.Tensor:
+    """The state matrix [dims, vdim] that one head's stored floats hold: element (d, col) with
+    d = 4 lanes r + 4 part + e lies at ((r * vdim + col) * lanes + part) * 4 + e, lanes = padded dims / 8."""
+    lanes = head_state.numel() // (8 * vdim)
+    return head_state.reshape(2, vdim, lanes, 4).permute(0, 2, 3, 1).reshape(8 * lanes, vdim)[:dims]
+
+
 def matrix_memory_aux_floats(dims: int, vdim: int) -> int:
     """Floats per head that ``matrix_memory`` keeps for the vector n and the running maximum m: a set
-    for every 32 columns of the state, each padded as the state's dims are, m after n."""
-    lanes = 1 if dims <= 32 else (2 if dims <= 64 else (4 if dims <= 128 else 8))
-    return -(-vdim // 32) * (32 * lanes + 4)
+    for every 16 columns of the state, each padded as the state's dims are, m after n."""
+    return -(-vdim // 16) * (matrix_memory_floats(dims, 1) + 4)
 
 
 def matrix_memory(q, k, v, in_logit, forget_logit, state, aux, cu_seqlens, seq_slot, y, heads, dim, vdim, cap, q_scale):
@@ -1832,7 +1844,7 @@ def matrix_memory(q, k, v, in_logit, forget_logit, state, aux, cu_seqlens, seq_s
     m' = max(f + m, i); S <- e^(f + m - m') S + e^(i - m') k v^T; n the same with k alone;
     y = S^T q / (max(|n . q|, e^(-m')) + 1e-6), q times ``q_scale``.  All inputs are slices of columns of
     one [T, *] tensor, q and k [T, heads * dim], v [T, heads * vdim], the logits [T, heads].  ``state``
-    [slots + 1, heads, recurrent_state_floats(dim, vdim)], ``aux`` [slots + 1, heads,
+    [slots + 1, heads, matrix_memory_floats(dim, vdim)] (see matrix_memory_matrix), ``aux`` [slots + 1, heads,
     matrix_memory_aux_floats(dim, vdim)], both zeros for a new sequence; dim up to 256."""
     _cuda(q, k, v, in_logit, forget_logit, state, aux, cu_seqlens, seq_slot, y)
     for t in (q, k, v, in_logit, forget_logit, state, aux, y):
@@ -1842,13 +1854,13 @@ def matrix_memory(q, k, v, in_logit, forget_logit, state, aux, cu_seqlens, seq_s
     assert all(c[1] == ld for c in cols) and y.is_contiguous() and y.shape[1] == heads * vdim
     assert q.shape[1] == k.shape[1] == heads * dim and v.shape[1] == heads * vdim
     assert in_logit.shape[1] == forget_logit.shape[1] == heads
-    assert state.is_contiguous() and tuple(state.shape[1:]) == (heads, recurrent_state_floats(dim, vdim))
+    assert state.is_contiguous() and tuple(state.shape[1:]) == (heads, matrix_memory_floats(dim, vdim))
     assert aux.is_contiguous() and tuple(aux.shape[1:]) == (heads, matrix_memory_aux_floats(dim, vdim))
     f = _fn("recurrent", "gb_matrix_memory",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-             c_int, c_int, c_int, c_float, c_float, c_void_p])
+             c_int, c_int, c_int, c_int, c_float, c_float, c_void_p])
     _check(f(*[c[0] for c in cols], ld, state.data_ptr(), aux.data_ptr(), cu_seqlens.data_ptr(), seq_slot.data_ptr(), y.data_ptr(),
-             seq_slot.numel(), heads, dim, vdim, float(cap or 0.0), q_scale, _stream()), "matrix_memory", "attention",
+             q.shape[0], seq_slot.numel(), heads, dim, vdim, float(cap or 0.0), q_scale, _stream()), "matrix_memory", "attention",
            _nbytes(q, k, v, y) + 2 * seq_slot.numel() * heads * dim * vdim * 4)
 
 

@@ -68,7 +68,7 @@ class MatrixMemory(Part):
         return kernels.gemm_units(self.compute) + [("recurrent", ())]
 
     def cache_needs(self):
-        return [StateNeed((self.heads, kernels.recurrent_state_floats(self.dim, self.vdim))),
+        return [StateNeed((self.heads, kernels.matrix_memory_floats(self.dim, self.vdim))),
                 StateNeed((self.heads, kernels.matrix_memory_aux_floats(self.dim, self.vdim)))]
 
     def weight_bytes(self):

@@ -194,6 +194,37 @@ for _name, (_n, _d) in NOGOSUN_PAIRS.items():
     PAIR_SHAPES[f"nogosun-{_name}"] = (f"Nogosun shape '{_name}'", _n)
 
 
+def mevuvik_shape(width, ff, heads, rank, q_rank, experts, top, vocab=102400):
+    """A Mevuvik config.json object of three layers, the second run twice: a two-branch layer of
+    attention without positions (half of ``heads`` heads of 128, an eighth as many kv heads as heads)
+    beside matrix memory (as many heads, keys of 64 and values of 128), experts behind it; a latent
+    attention layer of ``heads`` heads of 128 + 64 with values of 128, experts behind it; a two-branch
+    layer again, a dense feed-forward behind it.  A token passes ``ff`` hidden units in every layer."""
+    half = max(1, heads // 2)
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 2.0}, "expert": {"ff": ff // top}}
+    pair = {"left": {"heads": half, "kv_heads": max(1, heads // 8), "dim": 128, "vdim": 128, "scale": 128 ** -0.5},
+            "right": {"heads": half, "dim": 64, "vdim": 128, "gate_cap": 12.0}, "left_scale": 1.0, "right_scale": 1.0}
+    latent = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": rank, "scale": 192 ** -0.5,
+              "rot": {"base": 1000000.0, "dims": 64}}
+    return {"architecture": "Mevuvik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 1.0,
+            "logit_softcap": 30.0, "loop": {"start": 1, "stop": 2, "times": 2},
+            "layers": [{"type": "parallel", "mixer": pair, "mlp": moe},
+                       {"type": "latent_attention", "mixer": latent, "mlp": moe},
+                       {"type": "parallel", "mixer": pair, "mlp": {"kind": "dense", "ff": ff}}]}
+
+
+# Mevuvik beside Nogosun, the nearest design the package has (attention over every key beside a linear
+# recurrence, experts without gates, layers that run again): the same width, runs of layers, vocabulary,
+# heads, experts and hidden units a token passes.  Its latent attention's like is Toretar's ("toretar-*").
+MEVUVIK_PAIRS = {
+    "small": (mevuvik_shape(1024, 4096, 8, 256, 512, 16, 4), nogosun_shape(1024, 4096, 8, 512, 16, 4)),
+    "lite": (mevuvik_shape(2048, 8192, 16, 512, 1024, 32, 4), nogosun_shape(2048, 8192, 16, 1024, 32, 4)),
+    "mid": (mevuvik_shape(4096, 12288, 32, 512, 1536, 32, 4), nogosun_shape(4096, 12288, 32, 2048, 32, 4)),
+}
+for _name, (_m, _n) in MEVUVIK_PAIRS.items():
+    PAIR_SHAPES[f"mevuvik-{_name}"] = (f"Mevuvik shape '{_name}'", _m)
+
+
 def random_engine(cfg, max_batch, cache_tokens, options=""):
     """An engine over random weights of ``cfg`` made on the device; the tensors are taken out of
     their dict as they are bound, so that a model of 65 GB and its stacked q/k/v and gate/up copies
@@ -289,7 +320,8 @@ def timeline(shape, batch, context, layers, prompt, temperature, out=sys.stdout)
     from .sampling.sampler import BatchSampler, SamplingParams
     label, cfg = {**SHAPES, **PAIR_SHAPES}[shape]
     if "layers" in cfg:
-        cfg = dict(cfg, layers=cfg["layers"][:layers or len(cfg["layers"])])
+        if not cfg.get("loop"):           # a loop's layers are counted by their runs and kept whole
+            cfg = dict(cfg, layers=cfg["layers"][:layers or len(cfg["layers"])])
         n_layers, vocab = len(cfg["layers"]), cfg["vocab"]
     else:
         cfg = dict(cfg, num_hidden_layers=layers or cfg["num_hidden_layers"])
