@@ -325,3 +325,66 @@ NOGOSUN_C = {
         {"type": "attention", "mixer": _nogosun_attention(3, 1, 12, 0.3, 17, None, 50.0, 4), "mlp": _nogosun_moe(2, 1, 28)},
     ],
 }
+
+
+# ---------------------------------------------------------------------------------------------- Mevuvik
+def _mevuvik_latent(heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, base):
+    return {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": scale,
+            "rot": {"base": base, "dims": rot_dim}}
+
+
+def _mevuvik_pair(left, right, left_scale, right_scale):
+    lh, lg, ld, lv, lscale = left
+    rh, rd, rv, cap = right
+    return {"left": {"heads": lh, "kv_heads": lg, "dim": ld, "vdim": lv, "scale": lscale},
+            "right": {"heads": rh, "dim": rd, "vdim": rv, "gate_cap": cap}, "left_scale": left_scale, "right_scale": right_scale}
+
+
+def _mevuvik_moe(experts, top, ff, scale):
+    return {"kind": "moe", "router": {"experts": experts, "top": top, "scale": scale}, "expert": {"ff": ff}}
+
+
+def _mevuvik_dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+# Small sizes that no tensor-core attention takes but the products do (a width of 72): the first two
+# layers run twice, the loop's first layer being the model's first; a latent layer without feed-forward
+# inside the loop; three heads on one kv head; every expert chosen in one layer.
+MEVUVIK_A = {
+    "architecture": "Mevuvik", "vocab": 211, "width": 72, "norm": {"eps": 1e-5}, "residual_mult": 0.7, "logit_softcap": 9.0,
+    "loop": {"start": 0, "stop": 2, "times": 2},
+    "layers": [
+        {"type": "parallel", "mixer": _mevuvik_pair((3, 1, 20, 24, 0.25), (5, 24, 12, 6.0), 0.8, 1.3),
+         "mlp": _mevuvik_moe(5, 2, 40, 1.7)},
+        {"type": "latent_attention", "mixer": _mevuvik_latent(3, 24, 12, 20, 36, 44, 0.2, 500.0), "mlp": None},
+        {"type": "latent_attention", "mixer": _mevuvik_latent(2, 12, 8, 28, 20, 32, 0.3, 2e4), "mlp": _mevuvik_dense(56)},
+        {"type": "parallel", "mixer": _mevuvik_pair((4, 4, 12, 16, 0.35), (2, 40, 20, 20.0), 1.1, 0.6),
+         "mlp": _mevuvik_moe(3, 3, 24, 0.9)},
+    ],
+}
+
+# Sizes the tensor cores take: attention with keys of 64 and values of 128, latents of 112 + 16 (expanded
+# per head in long prompts) and of 64 + 32 (not expanded), matrix memory of 128 x 40; the last two layers
+# run three times, so that the loop ends with the model.
+MEVUVIK_B = {
+    "architecture": "Mevuvik", "vocab": 520, "width": 128, "norm": {"eps": 1e-6}, "residual_mult": 0.4, "logit_softcap": 25.0,
+    "loop": {"start": 1, "stop": 3, "times": 3},
+    "layers": [
+        {"type": "latent_attention", "mixer": _mevuvik_latent(6, 16, 16, 32, 64, 112, 0.18, 1e5), "mlp": _mevuvik_moe(8, 3, 64, 2.2)},
+        {"type": "parallel", "mixer": _mevuvik_pair((8, 2, 64, 128, 0.125), (2, 128, 40, 12.0), 0.9, 0.7), "mlp": _mevuvik_dense(192)},
+        {"type": "latent_attention", "mixer": _mevuvik_latent(4, 32, 32, 64, 40, 64, 0.125, 1e4), "mlp": _mevuvik_moe(6, 1, 96, 1.0)},
+    ],
+}
+
+# A width that is no multiple of 8 and heads that are no multiple of 16 (plain kernels throughout in
+# bfloat16): no loop, no cap on the logits, a residual factor and scales of one, a single kv head and a
+# single memory head, a single expert.
+MEVUVIK_C = {
+    "architecture": "Mevuvik", "vocab": 97, "width": 52, "norm": {"eps": 1e-6}, "residual_mult": 1.0, "logit_softcap": None,
+    "layers": [
+        {"type": "parallel", "mixer": _mevuvik_pair((1, 1, 12, 20, 0.3), (1, 20, 12, 1.5), 1.0, 1.0), "mlp": _mevuvik_moe(1, 1, 20, 1.0)},
+        {"type": "latent_attention", "mixer": _mevuvik_latent(1, 6, 10, 5, 9, 11, 0.25, 50.0), "mlp": _mevuvik_moe(4, 2, 12, 3.0)},
+        {"type": "parallel", "mixer": _mevuvik_pair((2, 1, 20, 12, 0.22), (3, 7, 9, 4.0), 1.0, 1.0), "mlp": None},
+    ],
+}
