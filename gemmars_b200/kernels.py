@@ -870,7 +870,8 @@ def latent_prepare(q_in, kv_in, g_in, norm_w, eps, inv_freq, rot, q_scale, q_nop
                    page_size, tok_pos, tok_seq, seq_slot, heads, dim, rd, rank, dense=None, half_layout=False):
     """From the float32 projections of a latent attention layer: the cache row of every token
     (RMS-normed latent ``kv_in[:, :rank]``, then the key part ``kv_in[:, rank:]`` with its first
-    ``rot`` dims rotated, as interleaved pairs or with ``half_layout`` as pairs (i, i + rot/2)) into the paged ``cache`` [pages, page_size, rank + rd];
+    ``rot`` dims rotated, as interleaved pairs or with ``half_layout`` as pairs (i, i + rot/2)) into
+    the paged ``cache`` [pages, page_size, rank + rd];
     the queries' unrotated dims times ``q_scale`` into ``q_nope`` [T, heads * dim], their rotated
     dims (rotated, scaled) into the last ``rd`` columns of each head of ``q_lat``
     [T, heads * (rank + rd)]; ``gate`` [T, heads] = sigmoid(g_in) (float32; None: no gate).  ``dense``
