@@ -5,12 +5,13 @@
 //
 //   gb_filter_rope_cache:  u [T, q | k | v] -> filter over time -> RMS norm of every q and k head
 //                          with a weight over its dims (when weights are given) -> rotation of the
-//                          first `rot` dims of every q and k head (dim i pairs with i + rot/2; angle
-//                          float(pos) * inv_freq[i], float32; cosines and sines times `rot_mag`) ->
-//                          q times 1 + qt_coef ln(floor((pos + 1) / qt_every) + 1) (when qt_every)
-//                          -> q rows, keys and values into pages.  With `v_from_k` the rows hold
-//                          q | k only and a value head is its key head as projected and filtered,
-//                          before norm and rotation
+//                          first `rot` dims of every q and k head (dim i pairs with i + rot/2, or with
+//                          `pairs` dim 2i with 2i + 1; angle float(pos) * inv_freq[i], float32; cosines
+//                          and sines times `rot_mag`) -> with `unit_after` every q and k head divided by
+//                          its root mean square (no weight) -> q times 1 + qt_coef ln(floor((pos + 1) /
+//                          qt_every) + 1) (when qt_every) -> q rows, keys and values into pages.  With
+//                          `v_from_k` the rows hold q | k only and a value head is its key head as
+//                          projected and filtered, before norm and rotation
 //   gb_attention_capped:   score = (q . k) * scale; score <- cap * tanh(score / cap) when cap > 0;
 //                          keys lo..p with lo = max(0, p + 1 - window), and with `keep_first` the
 //                          keys 0..keep_first-1 as well, wherever the window stands; softmax, whose
@@ -52,7 +53,7 @@ __global__ void __launch_bounds__(128) filter_rope_cache_kernel(
     const int* __restrict__ seq_slot, const int* __restrict__ cu, const int* __restrict__ page_table, int table_width,
     int page_size, T* __restrict__ q_out, long long ldq, T* __restrict__ kcache, T* __restrict__ vcache, int H, int G, int D,
     int Vd, const float* __restrict__ q_norm, const float* __restrict__ k_norm, float norm_eps, float rot_mag, float qt_coef,
-    int qt_every, int v_from_k) {
+    int qt_every, int v_from_k, int pairs, int unit_after) {
   __shared__ float vals[MAX_HEAD], cs[MAX_HEAD];   // cs: cos[rot / 2], then sin[rot / 2]
   __shared__ float scratch[33];
   pdl_release_next();
@@ -94,41 +95,56 @@ __global__ void __launch_bounds__(128) filter_rope_cache_kernel(
   }
   __syncthreads();
   const float temper = (hh < H && qt_every > 0) ? 1.0f + qt_coef * logf((float)((pos + 1) / qt_every + 1)) : 1.0f;
-  for (int i = threadIdx.x; i < D; i += blockDim.x) {
+  float turned[MAX_HEAD / 128], ss_after = 0.f;
+#pragma unroll
+  for (int u = 0; u < MAX_HEAD / 128; ++u) {
+    const int i = threadIdx.x + u * 128;
+    if (i >= D) break;
     float val = vals[i];
     if (i < rot) {
-      // the pair (a, b) = (dim j, dim j + half) becomes (a cos - b sin, b cos + a sin)
-      const int j = i < half ? i : i - half;
-      val = i < half ? val * cs[j] - vals[i + half] * cs[half + j] : val * cs[j] + vals[i - half] * cs[half + j];
+      // the pair (a, b) = (dim j, dim j + half), or (2j, 2j + 1), becomes (a cos - b sin, b cos + a sin)
+      const bool first = pairs ? (i & 1) == 0 : i < half;
+      const int j = pairs ? i >> 1 : (first ? i : i - half), step = pairs ? 1 : half;
+      val = first ? val * cs[j] - vals[i + step] * cs[half + j] : val * cs[j] + vals[i - step] * cs[half + j];
     }
-    if (hh < H) q_out[(size_t)t * ldq + hh * D + i] = from_f32<T>(val * temper);
-    else kcache[(((size_t)page * G + (hh - H)) * page_size + off) * D + i] = from_f32<T>(val);
+    turned[u] = val;
+    ss_after = fmaf(val, val, ss_after);
+  }
+  const float unit = unit_after ? 1.0f / sqrtf(block_sum(ss_after, scratch) / (float)D + norm_eps) : 1.0f;
+#pragma unroll
+  for (int u = 0; u < MAX_HEAD / 128; ++u) {
+    const int i = threadIdx.x + u * 128;
+    if (i >= D) break;
+    if (hh < H) q_out[(size_t)t * ldq + hh * D + i] = from_f32<T>(turned[u] * unit * temper);
+    else kcache[(((size_t)page * G + (hh - H)) * page_size + off) * D + i] = from_f32<T>(turned[u] * unit);
   }
 }
 
 // taps: [(H + G) D + G Vd, K] float32 (K = 0: no filter); state: [slots, K - 1, channels] float32.
 // G = 0: the rows hold queries only (a layer that reads another layer's keys and values).
-// q_norm, k_norm: float32 [D] or null; v_from_k needs Vd == D.
+// q_norm, k_norm: float32 [D] or null (norm_eps is theirs, or unit_after's: not both); v_from_k needs Vd == D.
 GB_EXPORT int gb_filter_rope_cache_ext(const void* u, int dtype, long long ldu, const float* taps, const float* state, int K,
                                        const float* inv_freq, int rot, const int* tok_pos, const int* tok_seq,
                                        const int* seq_slot, const int* cu, const int* page_table, int table_width,
                                        int page_size, void* q_out, long long ldq, void* kcache, void* vcache, int ntok, int H,
                                        int G, int D, int Vd, const float* q_norm, const float* k_norm, float norm_eps,
-                                       float rot_mag, float qt_coef, int qt_every, int v_from_k, cudaStream_t stream) {
+                                       float rot_mag, float qt_coef, int qt_every, int v_from_k, int pairs, int unit_after,
+                                       cudaStream_t stream) {
   if (ntok <= 0) return 0;
   if (K < 0 || K > MAX_TAPS || rot < 0 || rot > D || rot % 2 || H <= 0 || G < 0 || D <= 0 || D > MAX_HEAD || Vd <= 0)
     return GB_ERR_SIZE;
   if (v_from_k && (Vd != D || K > 1)) return GB_ERR_SIZE;
+  if (unit_after && (q_norm || k_norm)) return GB_ERR_ARG;
   if ((K > 0 && !taps) || (K > 1 && !state) || (rot > 0 && !inv_freq) || qt_every < 0) return GB_ERR_ARG;
   const dim3 grid(ntok, H + 2 * G);
   if (dtype == GB_F32)
     gb_launch(filter_rope_cache_kernel<float>, grid, 128, 0, stream, (const float*)u, ldu, taps, state, K, inv_freq, rot,
               tok_pos, tok_seq, seq_slot, cu, page_table, table_width, page_size, (float*)q_out, ldq, (float*)kcache,
-              (float*)vcache, H, G, D, Vd, q_norm, k_norm, norm_eps, rot_mag, qt_coef, qt_every, v_from_k);
+              (float*)vcache, H, G, D, Vd, q_norm, k_norm, norm_eps, rot_mag, qt_coef, qt_every, v_from_k, pairs, unit_after);
   else if (dtype == GB_BF16)
     gb_launch(filter_rope_cache_kernel<bf16>, grid, 128, 0, stream, (const bf16*)u, ldu, taps, state, K, inv_freq, rot,
               tok_pos, tok_seq, seq_slot, cu, page_table, table_width, page_size, (bf16*)q_out, ldq, (bf16*)kcache,
-              (bf16*)vcache, H, G, D, Vd, q_norm, k_norm, norm_eps, rot_mag, qt_coef, qt_every, v_from_k);
+              (bf16*)vcache, H, G, D, Vd, q_norm, k_norm, norm_eps, rot_mag, qt_coef, qt_every, v_from_k, pairs, unit_after);
   else
     return GB_ERR_DTYPE;
   return gb_launch_status();
@@ -141,7 +157,7 @@ GB_EXPORT int gb_filter_rope_cache(const void* u, int dtype, long long ldu, cons
                                    cudaStream_t stream) {
   return gb_filter_rope_cache_ext(u, dtype, ldu, taps, state, K, inv_freq, rot, tok_pos, tok_seq, seq_slot, cu, page_table,
                                   table_width, page_size, q_out, ldq, kcache, vcache, ntok, H, G, D, Vd, nullptr, nullptr, 0.f,
-                                  1.f, 0.f, 0, 0, stream);
+                                  1.f, 0.f, 0, 0, 0, 0, stream);
 }
 
 // One block per (token, query head); online softmax over chunks of 128 keys: first the kept keys

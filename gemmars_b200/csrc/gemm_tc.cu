@@ -846,14 +846,15 @@ constexpr int PERSISTENT_QKV_THREADS = 320, QKV_STAGING_BYTES = 65 * 1024;   // 
 // group; tile_expert[m tile] names it (-1: a tile no group uses, which every role skips) and the
 // tile's rows of W are the group's (W stacks the groups' matrices, rows_per_expert each).  The gated
 // mode then applies g = min(g, limit), u = clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + shift)
-// when limit > 0, and multiplies row r of the result by row_scale[r].  `act` (bfloat16 results of a
+// when limit > 0, and multiplies row r of the result by row_scale[r], or with `scale_in` row r of both sums
+// before the activation (an expert of the weighted input).  `act` (bfloat16 results of a
 // product without a gate, grouped or not): an activation of every result (out_act), then the row's scale.
 struct Grouped {
   const int* tile_expert = nullptr;
   const float* row_scale = nullptr;
   int rows_per_expert = 0;
   float limit = 0.f, alpha = 0.f, shift = 0.f;
-  int act = 0;
+  int act = 0, scale_in = 0;
 };
 __device__ __forceinline__ void act_rows(uint32_t (&v)[16], float bias, int act, const float* row_scale, int row, int M) {
 #pragma unroll
@@ -1086,13 +1087,22 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
             const uint32_t (&u)[16] = is_up ? v2 : got;
             const int row = m0 + c + (is_up ? 16 : 0);
             float r[16];
+            if (grp.scale_in) {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) r[j] = silu_mul(__uint_as_float(g[j]), __uint_as_float(u[j]));
-            if (grp.limit > 0.f) {
+              for (int j = 0; j < 16; ++j) {
+                const float sc = row + j < M ? grp.row_scale[row + j] : 0.f;
+                const float gs = __uint_as_float(g[j]) * sc, us = __uint_as_float(u[j]) * sc;
+                r[j] = grp.limit > 0.f ? clamped_gate(gs, us, grp) : silu_mul(gs, us);
+              }
+            } else {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) r[j] = silu_mul(__uint_as_float(g[j]), __uint_as_float(u[j]));
+            }
+            if (grp.limit > 0.f && !grp.scale_in) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) r[j] = clamped_gate(__uint_as_float(g[j]), __uint_as_float(u[j]), grp);
             }
-            if (grp.row_scale) {
+            if (grp.row_scale && !grp.scale_in) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) r[j] *= row + j < M ? grp.row_scale[row + j] : 0.f;
             }
@@ -1478,11 +1488,11 @@ GB_EXPORT int gb_gemm_tc_persistent(const void* x, const void* w, const float* b
 // group after the other, each group starting at a multiple of bn rows (M counts the padding);
 // w stacks `experts` matrices of N rows (2 N gated: gate rows, then up rows); tile_expert [M / bn].
 // mode 1: y float32 [M, N] = x W_g^T; mode 3: y bfloat16 [M, N] = row_scale * act(gate, up), act the
-// clamped form when limit > 0; mode 0: y bfloat16 [M, N] = row_scale * act(x W_g^T) (no gate rows in w;
+// clamped form when limit > 0, or with scale_in act(row_scale * gate, row_scale * up); mode 0: y bfloat16 [M, N] = row_scale * act(x W_g^T) (no gate rows in w;
 // act 1: the exact GELU, 2: the square of relu).  bn: 128 or 256.
 GB_EXPORT int gb_gemm_tc_grouped(const void* x, const void* w, void* y, int mode, int M, int N, int K, long long ldx,
                                  long long ldy, int bn, int ctas, int experts, const int* tile_expert, const float* row_scale,
-                                 float limit, float alpha, float shift, int act, cudaStream_t stream) {
+                                 float limit, float alpha, float shift, int act, int scale_in, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || experts <= 0) return 0;
   if (act < OUT_ACT_NONE || act > OUT_ACT_RELU2) return GB_ERR_ARG;
   if (K <= 0 || (K % 8) || (ldx % 8) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ctas <= 0) return GB_ERR_SIZE;
@@ -1495,6 +1505,7 @@ GB_EXPORT int gb_gemm_tc_grouped(const void* x, const void* w, void* y, int mode
   grp.rows_per_expert = N * (gated ? 2 : 1);
   grp.limit = limit; grp.alpha = alpha; grp.shift = shift;
   grp.act = mode == EPI_STORE_BF16 ? act : OUT_ACT_NONE;
+  grp.scale_in = gated && row_scale ? scale_in : 0;
   CUtensorMap mw, mx;
   if (!tensor_map(&mw, w, (uint64_t)experts * grp.rows_per_expert, (uint64_t)K, (uint64_t)K * 2, gated ? BM / 2 : BM)) return GB_ERR_ARG;
   if (!tensor_map(&mx, x, (uint64_t)M, (uint64_t)K, (uint64_t)ldx * 2, (uint32_t)bn)) return GB_ERR_ARG;

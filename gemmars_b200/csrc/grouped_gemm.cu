@@ -8,9 +8,12 @@
 //    features, so a thread holds both); the down product scales each row by its routing weight and
 //    leaves float32 rows that gb_moe_combine adds into the residual in slot order.  (Prompt steps
 //    run the same two products on the tcgen05 kernel of gemm_tc.cu instead, from a copy of the
-//    activations in a padded order: gb_moe_sort_padded, gb_moe_permute.)
+//    activations in a padded order: gb_moe_sort_padded, gb_moe_permute.)  With `scale_in` the routing
+//    weight multiplies the gate's and up's sums before the activation (an expert of the weighted input)
+//    and the down product scales nothing.
 //  * the per-head products of latent attention: group = head, every group has all the tokens,
-//    A and C rows are a token's slice of a wider row, with an optional scale per (token, head).
+//    A and C rows are a token's slice of a wider row, with an optional scale per (token, head) or an
+//    optional sigmoid gate per result.
 //
 // A CTA of 8 warps computes a tile of 128 rows x 128 columns (mma.sync m16n8k16, float32
 // accumulation), operands staged in shared memory by cp.async three blocks of 64 deep.  A CTA
@@ -35,6 +38,8 @@ struct GroupedArgs {
   int groups, rows, N, K;
   float limit, alpha, shift;                 // gated: g = min(g, limit), u = clamp(u, +-limit), g * sigmoid(alpha g) * (u + shift)
   int act;                                   // plain mode: an activation of every result before the scale (plain_act)
+  const float* gate; long long gate_rstride; long long gate_gstride;   // plain mode: times sigmoid(gate[row, column]), or null
+  int scale_in;                              // gated: the scale multiplies both sums before the activation, not the result
 };
 __device__ __forceinline__ float plain_act(float x, int act) {    // 1: the exact (erf) GELU; 2: the square of relu
   if (act == 2) return fmaxf(x, 0.f) * fmaxf(x, 0.f);
@@ -174,9 +179,10 @@ __global__ void __launch_bounds__(256, 2) grouped_gemm_kernel(GroupedArgs p) {
           for (int e = 0; e < 2; ++e) {
             const int f = n0 + (wn * 2 + (j >> 1)) * 8 + 2 * cq + e;
             if (f >= p.N) continue;
-            const float gt = fminf(acc[i][j][2 * half + e], p.limit);
-            const float up = fminf(fmaxf(acc[i][j + 1][2 * half + e], -p.limit), p.limit);
-            dst[f] = from_f32<TO>(gt / (1.0f + expf(-p.alpha * gt)) * (up + p.shift) * sc);
+            const float in = p.scale_in ? sc : 1.f;
+            const float gt = fminf(acc[i][j][2 * half + e] * in, p.limit);
+            const float up = fminf(fmaxf(acc[i][j + 1][2 * half + e] * in, -p.limit), p.limit);
+            dst[f] = from_f32<TO>(gt / (1.0f + expf(-p.alpha * gt)) * (up + p.shift) * (p.scale_in ? 1.f : sc));
           }
       } else {
 #pragma unroll
@@ -185,6 +191,11 @@ __global__ void __launch_bounds__(256, 2) grouped_gemm_kernel(GroupedArgs p) {
           float x = acc[i][j][2 * half], y = acc[i][j][2 * half + 1];
           if (p.act) { x = plain_act(x, p.act); y = plain_act(y, p.act); }
           x *= sc; y *= sc;
+          if (p.gate && col < p.N) {
+            const float* z = p.gate + crow * p.gate_rstride + (long long)g * p.gate_gstride + col;
+            x *= 1.0f / (1.0f + __expf(-z[0]));
+            if (col + 1 < p.N) y *= 1.0f / (1.0f + __expf(-z[1]));
+          }
           if (col + 1 < p.N && ((uintptr_t)(dst + col) & (2 * sizeof(TO) - 1)) == 0) {
             store2(dst + col, x, y);
           } else {
@@ -279,18 +290,19 @@ __global__ void __launch_bounds__(128) moe_permute_kernel(const bf16* __restrict
   if (threadIdx.x == 0) scale[r] = wts[e];
 }
 
-// residual[t] += col_scale (null: ones) * the sum over the token's slots, in slot order, of the rows the
-// down product left
+// residual[t] += (with `store`: =) col_scale (null: ones) * the sum over the token's slots, in slot order, of
+// the rows the down product left
 __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ place,
                                                           float* __restrict__ residual, long long ldr, int width, int top,
-                                                          const float* __restrict__ col_scale) {
+                                                          const float* __restrict__ col_scale, int store) {
   pdl_release_next();
   pdl_wait_prior();
   const int t = blockIdx.x;
   for (int n = threadIdx.x; n < width; n += 256) {
     float total = 0.f;
     for (int k = 0; k < top; ++k) total += rows[(size_t)place[(size_t)t * top + k] * width + n];
-    residual[(size_t)t * ldr + n] += col_scale ? total * col_scale[n] : total;
+    if (col_scale) total *= col_scale[n];
+    residual[(size_t)t * ldr + n] = store ? total : residual[(size_t)t * ldr + n] + total;
   }
 }
 
@@ -333,13 +345,15 @@ GB_EXPORT int gb_grouped_gemm(const void* a, long long lda, long long a_gstride,
                               const void* w, long long w_gstride, void* c, long long ldc, long long c_gstride,
                               const float* scale, const int* scale_rows, long long s_rstride, long long s_gstride,
                               const int* offsets, int groups, int rows, int max_rows, int N, int K, int gated, int out_f32,
-                              float limit, float alpha, float shift, cudaStream_t stream) {
+                              float limit, float alpha, float shift, const float* gate, long long gate_rstride,
+                              long long gate_gstride, int scale_in, cudaStream_t stream) {
   if (groups <= 0 || N <= 0 || max_rows <= 0) return 0;
   if (K <= 0 || K % 8 || lda % 8 || a_gstride % 8 || w_gstride % 8 || ((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return GB_ERR_SIZE;
   if (gated == 1 && out_f32) return GB_ERR_DTYPE;
-  if (gated < 0 || gated > 3) return GB_ERR_ARG;
+  if (gated < 0 || gated > 3 || (gate && gated == 1) || (scale_in && gated != 1)) return GB_ERR_ARG;
   GroupedArgs p{(const bf16*)a, lda, a_gstride, a_rows, a_div > 0 ? a_div : 1, (const bf16*)w, w_gstride, c, ldc, c_gstride,
-                scale, scale_rows, s_rstride, s_gstride, offsets, groups, rows, N, K, limit, alpha, shift, gated >= 2 ? gated - 1 : 0};
+                scale, scale_rows, s_rstride, s_gstride, offsets, groups, rows, N, K, limit, alpha, shift, gated >= 2 ? gated - 1 : 0, gate,
+                gate_rstride, gate_gstride, scale_in};
   const int row_tiles = offsets ? (max_rows + BM - 1) / BM + groups : groups * ((rows + BM - 1) / BM);
   if (gated == 1) return launch_grouped<MODE_GATED, bf16>(p, row_tiles, stream);
   if (out_f32) return launch_grouped<MODE_PLAIN, float>(p, row_tiles, stream);
@@ -373,9 +387,10 @@ GB_EXPORT int gb_moe_permute(const void* h, long long ldh, const int* row_entry,
 }
 
 GB_EXPORT int gb_moe_combine(const float* rows, const int* place, float* residual, long long ldr, int ntok, int width, int top,
-                             const float* col_scale, cudaStream_t stream) {
+                             const float* col_scale, int store, cudaStream_t stream) {
   if (ntok <= 0) return 0;
-  gb_launch(moe_combine_kernel, dim3(ntok), dim3(256), 0, stream, rows, place, residual, ldr, width, top, col_scale);
+  gb_launch(moe_combine_kernel, dim3(ntok), dim3(256), 0, stream, rows, place, residual, ldr, width, top, col_scale,
+            store);
   return gb_launch_status();
 }
 

@@ -10,7 +10,8 @@
 //   s[t, h, j]      = qa[t, h] . row[j]           (q already carries the score scale)
 //   p               = softmax_j over j <= pos(t)  (float32)
 //   ol[t, h]        = sum_j p[j] row[j, :rank]
-//   o[t, h]         = gate[t, h] * W_uv[h] ol[t, h]   (gb_heads_gemm with a row scale)
+//   o[t, h]         = gate[t, h] * W_uv[h] ol[t, h]   (gb_heads_gemm with a row scale), or with a gate per
+//                    output number  sigmoid(z[t, h, :]) * W_uv[h] ol[t, h]
 //
 // This unit holds what every precision and size can use: the kernel that norms, rotates and
 // writes the cache row (gb_latent_prepare), the per-head products (gb_heads_gemm, FFMA), the
@@ -20,10 +21,12 @@
 #include "common.cuh"
 
 // Rotation of a pair (u, v) -> (u cos - v sin, v cos + u sin), angle = float(pos) * inv_freq[i], all in
-// float32.  Pair i < rot/2 is dims (2i, 2i+1), or with the half layout (i, i + rot/2).
-__device__ __forceinline__ void rotate_pair(float u, float v, float angle, float& ou, float& ov) {
+// float32, cosine and sine times `mag`.  Pair i < rot/2 is dims (2i, 2i+1), or with the half layout (i, i + rot/2).
+__device__ __forceinline__ void rotate_pair(float u, float v, float angle, float mag, float& ou, float& ov) {
   float s, c;
   sincosf(angle, &s, &c);
+  s *= mag;
+  c *= mag;
   ou = u * c - v * s;
   ov = v * c + u * s;
 }
@@ -37,7 +40,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
     T* __restrict__ q_lat, long long ldql, float* __restrict__ gate, T* __restrict__ cache,
     const int* __restrict__ page_table, int table_width, int page_size, const int* __restrict__ tok_pos,
     const int* __restrict__ tok_seq, const int* __restrict__ seq_slot, int H, int dim, int rd, int rank,
-    T* __restrict__ dense, long long ldd, int half_layout) {
+    T* __restrict__ dense, long long ldd, int half_layout, float rot_mag) {
   __shared__ float scratch[34];
   pdl_release_next();
   pdl_wait_prior();
@@ -69,7 +72,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
       const int a = turns && half_layout ? i : 2 * i, b = turns && half_layout ? i + rot / 2 : 2 * i + 1;
       if (turns) {
         float u, v;
-        rotate_pair(kv[rank + a], kv[rank + b], fpos * inv_freq[i], u, v);
+        rotate_pair(kv[rank + a], kv[rank + b], fpos * inv_freq[i], rot_mag, u, v);
         row[rank + a] = from_f32<T>(u);
         row[rank + b] = from_f32<T>(v);
       } else {
@@ -94,7 +97,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
     T* dst = q_lat + (size_t)t * ldql + (size_t)h * (rank + rd) + rank;
     if (turns) {
       float u, v;
-      rotate_pair(src[a], src[b], fpos * inv_freq[i], u, v);
+      rotate_pair(src[a], src[b], fpos * inv_freq[i], rot_mag, u, v);
       dst[a] = from_f32<T>(u * q_scale);
       dst[b] = from_f32<T>(v * q_scale);
     } else {
@@ -111,14 +114,15 @@ GB_EXPORT int gb_latent_prepare(const float* q_in, long long ldq, const float* k
                                 float q_scale, void* q_nope, long long ldqn, void* q_lat, long long ldql, float* gate,
                                 void* cache, int dtype, const int* page_table, int table_width, int page_size,
                                 const int* tok_pos, const int* tok_seq, const int* seq_slot, int ntok, int H, int dim,
-                                int rd, int rank, void* dense, long long ldd, int half_layout, cudaStream_t stream) {
+                                int rd, int rank, void* dense, long long ldd, int half_layout, float rot_mag,
+                                cudaStream_t stream) {
   if (ntok <= 0) return 0;
   if (H <= 0 || dim < 0 || rd < 0 || rank <= 0 || rot < 0 || rot > rd || (rot & 1)) return GB_ERR_SIZE;
   if (rot > 0 && inv_freq == nullptr) return GB_ERR_ARG;
 #define LAUNCH(T)                                                                                                     \
   gb_launch(latent_prepare_kernel<T>, dim3(ntok), dim3(256), 0, stream, q_in, ldq, kv_in, ldkv, g_in, ldg, norm_w, eps, \
             inv_freq, rot, q_scale, (T*)q_nope, ldqn, (T*)q_lat, ldql, gate, (T*)cache, page_table, table_width,       \
-            page_size, tok_pos, tok_seq, seq_slot, H, dim, rd, rank, (T*)dense, ldd, half_layout)
+            page_size, tok_pos, tok_seq, seq_slot, H, dim, rd, rank, (T*)dense, ldd, half_layout, rot_mag)
   if (dtype == GB_F32) LAUNCH(float);
   else if (dtype == GB_BF16) LAUNCH(bf16);
   else return GB_ERR_DTYPE;
@@ -128,14 +132,15 @@ GB_EXPORT int gb_latent_prepare(const float* q_in, long long ldq, const float* k
 
 // ---------------------------------------------------------------------------------------------
 // y[t, h, n] = scale[t, h] * sum_k x[t, h, k] * w[h, n, k]: one product per head, FFMA with
-// float32 accumulation in ascending k (a row's result does not depend on the other rows).
+// float32 accumulation in ascending k (a row's result does not depend on the other rows).  With `gate`
+// (rows ldg apart, head h's numbers from h * N) the result is multiplied by sigmoid(gate[t, h * N + n]).
 constexpr int HB = 64, HK = 16;
 
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256) heads_gemm_kernel(const TI* __restrict__ x, long long ldx_t, long long ldx_h,
                                                          const TI* __restrict__ w, TO* __restrict__ y, long long ldy_t,
                                                          long long ldy_h, const float* __restrict__ scale, int M, int H,
-                                                         int N, int K) {
+                                                         int N, int K, const float* __restrict__ gate, long long ldg) {
   pdl_release_next();
   pdl_wait_prior();
   __shared__ float xs[HK][HB + 4];
@@ -176,23 +181,25 @@ __global__ void __launch_bounds__(256) heads_gemm_kernel(const TI* __restrict__ 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int gn = n0 + tn + j;
-      if (gn < N) y[(size_t)gm * ldy_t + (size_t)h * ldy_h + gn] = from_f32<TO>(acc[i][j] * s);
+      if (gn >= N) continue;
+      const float open = gate ? 1.0f / (1.0f + expf(-gate[(size_t)gm * ldg + (size_t)h * N + gn])) : 1.f;
+      y[(size_t)gm * ldy_t + (size_t)h * ldy_h + gn] = from_f32<TO>(acc[i][j] * s * open);
     }
   }
 }
 
 GB_EXPORT int gb_heads_gemm(const void* x, long long ldx_t, long long ldx_h, const void* w, void* y, long long ldy_t,
                             long long ldy_h, const float* scale, int dtype, int M, int H, int N, int K,
-                            cudaStream_t stream) {
+                            const float* gate, long long ldg, cudaStream_t stream) {
   if (M <= 0 || H <= 0 || N <= 0) return 0;
   if (K <= 0 || H > 65535) return GB_ERR_SIZE;
   dim3 grid((N + HB - 1) / HB, (M + HB - 1) / HB, H);
   if (dtype == GB_F32)
     gb_launch(heads_gemm_kernel<float, float>, grid, dim3(256), 0, stream, (const float*)x, ldx_t, ldx_h, (const float*)w,
-              (float*)y, ldy_t, ldy_h, scale, M, H, N, K);
+              (float*)y, ldy_t, ldy_h, scale, M, H, N, K, gate, ldg);
   else if (dtype == GB_BF16)
     gb_launch(heads_gemm_kernel<bf16, bf16>, grid, dim3(256), 0, stream, (const bf16*)x, ldx_t, ldx_h, (const bf16*)w,
-              (bf16*)y, ldy_t, ldy_h, scale, M, H, N, K);
+              (bf16*)y, ldy_t, ldy_h, scale, M, H, N, K, gate, ldg);
   else
     return GB_ERR_DTYPE;
   return gb_launch_status();
@@ -293,7 +300,7 @@ GB_EXPORT int gb_latent_attention_ref(const void* qa, long long ldq, void* out, 
 // of every head.
 template <typename T>
 __global__ void rope_pairs_kernel(T* __restrict__ x, long long ldx, const int* __restrict__ tok_pos,
-                                  const float* __restrict__ inv_freq, int heads, int hd, int rot) {
+                                  const float* __restrict__ inv_freq, int heads, int hd, int rot, float mag) {
   pdl_release_next();
   pdl_wait_prior();
   const int t = blockIdx.x;
@@ -303,20 +310,20 @@ __global__ void rope_pairs_kernel(T* __restrict__ x, long long ldx, const int* _
     const int h = e / half, i = e % half;
     T* v = x + (size_t)t * ldx + (size_t)h * hd + 2 * i;
     float a, b;
-    rotate_pair(to_f32(v[0]), to_f32(v[1]), fpos * inv_freq[i], a, b);
+    rotate_pair(to_f32(v[0]), to_f32(v[1]), fpos * inv_freq[i], mag, a, b);
     v[0] = from_f32<T>(a);
     v[1] = from_f32<T>(b);
   }
 }
 
 GB_EXPORT int gb_rope_pairs(void* x, long long ldx, int dtype, const int* tok_pos, const float* inv_freq, int ntok,
-                            int heads, int hd, int rot, cudaStream_t stream) {
+                            int heads, int hd, int rot, float mag, cudaStream_t stream) {
   if (ntok <= 0 || rot <= 0) return 0;
   if (rot > hd || (rot & 1)) return GB_ERR_SIZE;
   if (dtype == GB_F32)
-    gb_launch(rope_pairs_kernel<float>, dim3(ntok), dim3(128), 0, stream, (float*)x, ldx, tok_pos, inv_freq, heads, hd, rot);
+    gb_launch(rope_pairs_kernel<float>, dim3(ntok), dim3(128), 0, stream, (float*)x, ldx, tok_pos, inv_freq, heads, hd, rot, mag);
   else if (dtype == GB_BF16)
-    gb_launch(rope_pairs_kernel<bf16>, dim3(ntok), dim3(128), 0, stream, (bf16*)x, ldx, tok_pos, inv_freq, heads, hd, rot);
+    gb_launch(rope_pairs_kernel<bf16>, dim3(ntok), dim3(128), 0, stream, (bf16*)x, ldx, tok_pos, inv_freq, heads, hd, rot, mag);
   else
     return GB_ERR_DTYPE;
   return gb_launch_status();

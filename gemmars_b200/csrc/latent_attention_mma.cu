@@ -23,7 +23,8 @@
 // The same kernel serves a prompt step whose keys and values were expanded per head (rows
 // [v | k_nope | k_rot] with the value's width in RANK's place): head_stride > 0 gives every head rows
 // of its own, contiguous from a sequence's first packed token, one head per grid layer, and
-// out_scale (the layer's gate) is multiplied into the output.
+// out_scale (the layer's gate per head) or sigmoid(out_gate) (one per output number) is multiplied into
+// the output.
 #include "mma.cuh"
 
 #ifndef GB_LATENT_RANK
@@ -72,7 +73,8 @@ latent_attention_mma_kernel(const bf16* __restrict__ qa, long long ldq, bf16* __
                             float* __restrict__ part, const bf16* __restrict__ cache, const int* __restrict__ page_table,
                             int table_width, int page_size, const int* __restrict__ cu_seqlens,
                             const int* __restrict__ seq_start, const int* __restrict__ seq_slot, int n_seqs, int H,
-                            int window, int ksplits, long long head_stride, const float* __restrict__ out_scale) {
+                            int window, int ksplits, long long head_stride, const float* __restrict__ out_scale,
+                            const float* __restrict__ out_gate, long long ldg) {
   constexpr int NB = KEYS / 8;                         // blocks of 8 keys a tile
   constexpr int SXP = KEYS + 4;                        // pitch of the exchanged scores
   static_assert(NB % 2 == 0, "key blocks come in pairs");
@@ -276,6 +278,14 @@ latent_attention_mma_kernel(const bf16* __restrict__ qa, long long ldq, bf16* __
       float inv = 1.0f / (half ? l1 : l0);
       if (out_scale) inv *= out_scale[(size_t)(tok_base + row / H) * heads_all + (per_head ? hz : row % H)];
       bf16* dst = out + (size_t)(tok_base + row / H) * ldo + (size_t)(row % H) * RANK + w * DW + 2 * c;
+      if (out_gate) {
+        const float* z = out_gate + (size_t)(tok_base + row / H) * ldg + (size_t)(per_head ? hz : row % H) * RANK + w * DW + 2 * c;
+#pragma unroll
+        for (int d = 0; d < DW / 8; ++d)
+          *(uint32_t*)(dst + d * 8) = pack_bf16(o[d][2 * half] * inv / (1.0f + __expf(-z[d * 8])),
+                                                o[d][2 * half + 1] * inv / (1.0f + __expf(-z[d * 8 + 1])));
+        continue;
+      }
 #pragma unroll
       for (int d = 0; d < DW / 8; ++d) *(uint32_t*)(dst + d * 8) = pack_bf16(o[d][2 * half] * inv, o[d][2 * half + 1] * inv);
     }
@@ -331,7 +341,7 @@ template <int KEYS>
 int launch_latent(const bf16* qa, long long ldq, bf16* out, long long ldo, float* part, const bf16* cache, const int* page_table,
                   int table_width, int page_size, const int* cu_seqlens, const int* seq_start, const int* seq_slot, int n_seqs,
                   int ntok, int H, int groups, int window, int ksplits, long long head_stride, const float* out_scale,
-                  cudaStream_t stream) {
+                  const float* out_gate, long long ldg, cudaStream_t stream) {
   const int tile_rows = groups * 16;
   if (tile_rows > 2 * KEYS) return GB_ERR_SIZE;       // the queries are staged in the key buffers
   const size_t smem = 2 * (size_t)KEYS * LDS * sizeof(bf16) +
@@ -346,7 +356,7 @@ int launch_latent(const bf16* qa, long long ldq, bf16* out, long long ldo, float
   dim3 grid(((long long)ntok * row_heads + tile_rows - 1) / tile_rows + n_seqs, ksplits, head_stride > 0 ? H : 1);
   gb_launch(latent_attention_mma_kernel<KEYS>, grid, dim3(groups * NSPLIT * 32), smem, stream, qa, ldq, out, ldo, part, cache,
             page_table, table_width, page_size, cu_seqlens, seq_start, seq_slot, n_seqs, H, window, ksplits, head_stride,
-            out_scale);
+            out_scale, out_gate, ldg);
   return 0;
 }
 
@@ -363,26 +373,28 @@ GB_EXPORT long long gb_latent_attention_mma_scratch(int ntok, int H, int ksplits
 // one sequence brings, for the size of a CTA.  head_stride > 0: the rows are per head and contiguous
 // (cache: [H][all packed tokens + a tile's worth][RANK + ROT], elements head_stride apart; every
 // sequence starts at position 0; no page table; ksplits 1).  out_scale: float32 [ntok, H] or null,
-// multiplied into the output (ksplits 1 only).
+// multiplied into the output (ksplits 1 only); out_gate: float32 [ntok, H * RANK] rows ldg apart or null, its
+// sigmoid multiplied into the output (ksplits 1 only).
 GB_EXPORT int gb_latent_attention_mma(const void* qa, long long ldq, void* out, long long ldo, float* part,
                                       const void* cache, const int* page_table, int table_width, int page_size,
                                       const int* cu_seqlens, const int* seq_start, const int* seq_slot, int n_seqs,
                                       int ntok, int H, int rank, int rot, int max_rows, int window, int ksplits,
-                                      long long head_stride, const float* out_scale, cudaStream_t stream) {
+                                      long long head_stride, const float* out_scale, const float* out_gate, long long ldg,
+                                      cudaStream_t stream) {
   if (ntok <= 0 || n_seqs <= 0) return 0;
   if (rank != RANK || rot != ROT || H <= 0 || page_size % 64 || ksplits < 1 || ksplits > MAX_KSPLITS) return GB_ERR_SIZE;
   if (((uintptr_t)qa & 15) || (ldq % 8) || ((uintptr_t)out & 3) || (ldo % 2) || ((uintptr_t)cache & 15)) return GB_ERR_SIZE;
-  if (ksplits > 1 && (part == nullptr || ((uintptr_t)part & 15) || head_stride > 0 || out_scale)) return GB_ERR_ARG;
+  if (ksplits > 1 && (part == nullptr || ((uintptr_t)part & 15) || head_stride > 0 || out_scale || out_gate)) return GB_ERR_ARG;
   if (head_stride > 0 && (H > 65535 || head_stride % 8)) return GB_ERR_SIZE;
   int groups = (max_rows + 15) / 16;
   groups = groups < 1 ? 1 : (groups > MAX_GROUPS ? MAX_GROUPS : groups);
   int rc;
   if (ksplits > 1)
     rc = launch_latent<32>((const bf16*)qa, ldq, (bf16*)out, ldo, part, (const bf16*)cache, page_table, table_width, page_size,
-                           cu_seqlens, seq_start, seq_slot, n_seqs, ntok, H, groups, window, ksplits, head_stride, out_scale, stream);
+                           cu_seqlens, seq_start, seq_slot, n_seqs, ntok, H, groups, window, ksplits, head_stride, out_scale, out_gate, ldg, stream);
   else
     rc = launch_latent<64>((const bf16*)qa, ldq, (bf16*)out, ldo, part, (const bf16*)cache, page_table, table_width, page_size,
-                           cu_seqlens, seq_start, seq_slot, n_seqs, ntok, H, groups, window, ksplits, head_stride, out_scale, stream);
+                           cu_seqlens, seq_start, seq_slot, n_seqs, ntok, H, groups, window, ksplits, head_stride, out_scale, out_gate, ldg, stream);
   if (rc) return rc;
   if (ksplits > 1)
     gb_launch(latent_attention_merge_kernel, dim3(ntok * H), dim3(128), 0, stream, (const float*)part, (bf16*)out, ldo, H,

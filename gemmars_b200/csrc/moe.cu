@@ -8,9 +8,12 @@
 //
 // Three more forms for designs that ask for them: ROUTE_SOFTMAX_ALL (the weights are the chosen experts'
 // shares of the softmax over ALL experts, not renormalized); ROUTE_SIGMOID (scores s = sigmoid(router . h);
-// chosen by s + bias, weighted by s / (sum of the chosen s + 1e-20) * scale, the bias left out); and
+// chosen by s + bias, weighted by s / (sum of the chosen s + 1e-20) * scale, the bias left out; in
+// ROUTE_SIGMOID_RAW by s * scale as it is); and
 // experts without a gate (gb_moe_up: y = act(up h), act the exact, erf GELU or the square of relu; out =
 // down y; the first matrices are [E, ff, width]).  `col_scale` [width] multiplies what is added into the residual.
+// A design may weigh an expert's input instead of its output, expert(weight * h): `in_wts` multiplies the
+// gate's and up's sums before the activation, and gb_moe_down is given no weights.
 //
 // The router's logits are a product like any other (the part computes them in float32); this unit
 // picks the experts from them and runs the experts token-major: a block owns one (token, chosen
@@ -74,7 +77,7 @@ template <typename T> __device__ __forceinline__ bool rows_vectorize(const T* ba
 // ---- router: the logits come from a product (float32 [ntok, ldz]); a warp per token adds the
 // bias, picks the `top` largest (the lower index wins a tie) and weighs them as `mode` says (the
 // softmax over those alone by default).  Column E of z, when there is one, is the shared expert's gate logit.
-enum { ROUTE_SOFTMAX_TOP = 0, ROUTE_SOFTMAX_ALL = 1, ROUTE_SIGMOID = 2 };
+enum { ROUTE_SOFTMAX_TOP = 0, ROUTE_SOFTMAX_ALL = 1, ROUTE_SIGMOID = 2, ROUTE_SIGMOID_RAW = 3 };
 __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__ zin, long long ldz,
                                                        const float* __restrict__ bias, int* __restrict__ idx,
                                                        float* __restrict__ wts, float* __restrict__ sg, int ntok, int E,
@@ -88,7 +91,7 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__
   float* z = smem + (size_t)warp * E;
   for (int e = lane; e < E; e += 32) {
     const float v = zin[(size_t)t * ldz + e];
-    z[e] = (mode == ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-v)) : v) + (bias ? bias[e] : 0.f);
+    z[e] = (mode >= ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-v)) : v) + (bias ? bias[e] : 0.f);
   }
   if (has_gate && lane == 0) sg[t] = 1.0f / (1.0f + expf(-zin[(size_t)t * ldz + E]));
   __syncwarp();
@@ -115,9 +118,9 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__
     }
     __syncwarp();
   }
-  if (mode == ROUTE_SIGMOID) {
+  if (mode >= ROUTE_SIGMOID) {
     const float s = lane < top ? 1.0f / (1.0f + expf(-zin[(size_t)t * ldz + mine_at])) : 0.f;
-    const float total = warp_sum(s) + 1e-20f;
+    const float total = mode == ROUTE_SIGMOID ? warp_sum(s) + 1e-20f : 1.f;
     if (lane < top) wts[(size_t)t * top + lane] = s / total * scale;
     return;
   }
@@ -139,7 +142,8 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(const T* __restrict__ 
                                                           const int* __restrict__ idx, const T* __restrict__ w_gu,
                                                           const T* __restrict__ ws_gu, T* __restrict__ y, int width,
                                                           int ff, int ffs, int ffmax, int top, int slots, float limit,
-                                                          float limit_s, float alpha, float shift) {
+                                                          float limit_s, float alpha, float shift,
+                                                          const float* __restrict__ in_wts) {
   extern __shared__ float xs[];   // [width]
   pdl_release_next();
   pdl_wait_prior();
@@ -160,6 +164,11 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(const T* __restrict__ 
     g = warp_sum(g);
     u = warp_sum(u);
     if (lane == 0) {
+      if (in_wts && routed) {
+        const float wt = in_wts[(size_t)t * top + s];
+        g *= wt;
+        u *= wt;
+      }
       g = fminf(g, lim);
       u = fminf(fmaxf(u, -lim), lim);
       const float a = g / (1.0f + expf(-alpha * g)) * (u + shift);
@@ -220,7 +229,7 @@ __global__ void __launch_bounds__(256) moe_down_kernel(const T* __restrict__ y, 
   for (int i = tid; i < nf; i += 256) ys[i] = to_f32(y[((size_t)t * slots + s) * ffmax + i]);
   __syncthreads();
   const T* W = routed ? w_d + (size_t)idx[(size_t)t * top + s] * width * ff : ws_d;
-  const float wt = routed ? wts[(size_t)t * top + s] : sg[t];
+  const float wt = routed ? (wts ? wts[(size_t)t * top + s] : 1.f) : sg[t];
   const bool vec = rows_vectorize(W, nf);
   const int n0 = blockIdx.y * FEATS;
   for (int n = n0 + warp * 2; n < min(width, n0 + FEATS); n += 16) {
@@ -238,21 +247,22 @@ __global__ void __launch_bounds__(256) moe_down_kernel(const T* __restrict__ y, 
 
 __global__ void __launch_bounds__(256) moe_sum_kernel(const float* __restrict__ rows, float* __restrict__ residual,
                                                       long long ldr, int width, int slots,
-                                                      const float* __restrict__ col_scale) {
+                                                      const float* __restrict__ col_scale, int store) {
   pdl_release_next();
   pdl_wait_prior();
   const int t = blockIdx.x;
   for (int n = blockIdx.y * 256 + threadIdx.x; n < width; n += gridDim.y * 256) {
     float total = 0.f;
     for (int s = 0; s < slots; ++s) total += rows[((size_t)t * slots + s) * width + n];
-    residual[(size_t)t * ldr + n] += col_scale ? total * col_scale[n] : total;
+    if (col_scale) total *= col_scale[n];
+    residual[(size_t)t * ldr + n] = store ? total : residual[(size_t)t * ldr + n] + total;
   }
 }
 
 GB_EXPORT int gb_moe_topk_mode(const float* z, long long ldz, const float* bias, int* idx, float* wts, float* sg, int ntok,
                                int E, int top, int has_gate, int mode, float scale, cudaStream_t stream) {
   if (ntok <= 0) return 0;
-  if (mode < ROUTE_SOFTMAX_TOP || mode > ROUTE_SIGMOID) return GB_ERR_ARG;
+  if (mode < ROUTE_SOFTMAX_TOP || mode > ROUTE_SIGMOID_RAW) return GB_ERR_ARG;
   if (E <= 0 || top <= 0 || top > 32 || top > E || E > 2048) return GB_ERR_SIZE;
   gb_launch(moe_topk_kernel, dim3((ntok + 3) / 4), dim3(128), (size_t)4 * E * sizeof(float), stream, z, ldz, bias, idx, wts, sg,
             ntok, E, top, has_gate, mode, scale);
@@ -265,10 +275,11 @@ GB_EXPORT int gb_moe_topk(const float* z, long long ldz, const float* bias, int*
 }
 
 // w_gu: [E, 2 ff, width] (an expert's gate rows, then its up rows); ws_gu: [2 ffs, width] or null;
-// y: [ntok, slots, ffmax], slots = top (+ 1 with a shared expert), ffmax = max(ff, ffs).
+// y: [ntok, slots, ffmax], slots = top (+ 1 with a shared expert), ffmax = max(ff, ffs).  in_wts: float32
+// [ntok, top], factors on the routed experts' inputs, or null.
 GB_EXPORT int gb_moe_gate_up(const void* h, long long ldh, int dtype, const int* idx, const void* w_gu, const void* ws_gu,
                              void* y, int ntok, int width, int ff, int ffs, int top, float limit, float limit_s,
-                             float alpha, float shift, cudaStream_t stream) {
+                             float alpha, float shift, const float* in_wts, cudaStream_t stream) {
   if (ntok <= 0) return 0;
   const int slots = top + (ws_gu ? 1 : 0), ffmax = ff > ffs ? ff : ffs;
   if (width <= 0 || ffmax <= 0 || slots <= 0) return GB_ERR_SIZE;
@@ -277,10 +288,10 @@ GB_EXPORT int gb_moe_gate_up(const void* h, long long ldh, int dtype, const int*
   dim3 grid(ntok * slots, (ffmax + FEATS - 1) / FEATS);
   if (dtype == GB_F32)
     gb_launch(moe_gate_up_kernel<float>, grid, dim3(256), smem, stream, (const float*)h, ldh, idx, (const float*)w_gu,
-              (const float*)ws_gu, (float*)y, width, ff, ffs, ffmax, top, slots, limit, limit_s, alpha, shift);
+              (const float*)ws_gu, (float*)y, width, ff, ffs, ffmax, top, slots, limit, limit_s, alpha, shift, in_wts);
   else if (dtype == GB_BF16)
     gb_launch(moe_gate_up_kernel<bf16>, grid, dim3(256), smem, stream, (const bf16*)h, ldh, idx, (const bf16*)w_gu,
-              (const bf16*)ws_gu, (bf16*)y, width, ff, ffs, ffmax, top, slots, limit, limit_s, alpha, shift);
+              (const bf16*)ws_gu, (bf16*)y, width, ff, ffs, ffmax, top, slots, limit, limit_s, alpha, shift, in_wts);
   else
     return GB_ERR_DTYPE;
   return gb_launch_status();
@@ -307,10 +318,10 @@ GB_EXPORT int gb_moe_up(const void* h, long long ldh, int dtype, const int* idx,
 }
 
 // w_d: [E, width, ff]; ws_d: [width, ffs] or null; rows: float32 scratch [ntok, slots, width];
-// residual: float32 [ntok, width] rows ldr apart.
+// residual: float32 [ntok, width] rows ldr apart, added to, or with `store` written.  wts: null: ones.
 GB_EXPORT int gb_moe_down(const void* y, int dtype, const int* idx, const float* wts, const float* sg, const void* w_d,
                           const void* ws_d, float* rows, float* residual, long long ldr, int ntok, int width, int ff, int ffs,
-                          int top, const float* col_scale, cudaStream_t stream) {
+                          int top, const float* col_scale, int store, cudaStream_t stream) {
   if (ntok <= 0) return 0;
   const int slots = top + (ws_d ? 1 : 0), ffmax = ff > ffs ? ff : ffs;
   if (width <= 0 || ffmax <= 0 || slots <= 0) return GB_ERR_SIZE;
@@ -326,6 +337,6 @@ GB_EXPORT int gb_moe_down(const void* y, int dtype, const int* idx, const float*
   else
     return GB_ERR_DTYPE;
   gb_launch(moe_sum_kernel, dim3(ntok, (width + 1023) / 1024), dim3(256), 0, stream, (const float*)rows, residual, ldr, width,
-            slots, col_scale);
+            slots, col_scale, store);
   return gb_launch_status();
 }

@@ -867,11 +867,12 @@ def attention_prefill_tc_status(head_dim: int = 0, reset: bool = True) -> int:
 # --------------------------------------------------------------------------- latent attention
 
 def latent_prepare(q_in, kv_in, g_in, norm_w, eps, inv_freq, rot, q_scale, q_nope, q_lat, gate, cache, page_table,
-                   page_size, tok_pos, tok_seq, seq_slot, heads, dim, rd, rank, dense=None, half_layout=False):
+                   page_size, tok_pos, tok_seq, seq_slot, heads, dim, rd, rank, dense=None, half_layout=False,
+                   rot_magnitude: float = 1.0):
     """From the float32 projections of a latent attention layer: the cache row of every token
     (RMS-normed latent ``kv_in[:, :rank]``, then the key part ``kv_in[:, rank:]`` with its first
-    ``rot`` dims rotated, as interleaved pairs or with ``half_layout`` as pairs (i, i + rot/2)) into
-    the paged ``cache`` [pages, page_size, rank + rd];
+    ``rot`` dims rotated, as interleaved pairs or with ``half_layout`` as pairs (i, i + rot/2), cosines
+    and sines times ``rot_magnitude``) into the paged ``cache`` [pages, page_size, rank + rd];
     the queries' unrotated dims times ``q_scale`` into ``q_nope`` [T, heads * dim], their rotated
     dims (rotated, scaled) into the last ``rd`` columns of each head of ``q_lat``
     [T, heads * (rank + rd)]; ``gate`` [T, heads] = sigmoid(g_in) (float32; None: no gate).  ``dense``
@@ -892,7 +893,7 @@ def latent_prepare(q_in, kv_in, g_in, norm_w, eps, inv_freq, rot, q_scale, q_nop
     f = _fn("latent_attention", "gb_latent_prepare",
             [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_float,
              c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
-             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p])
+             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_int, c_float, c_void_p])
     if dense is not None:
         assert dense.dtype == q_lat.dtype and dense.shape == (t, rank + rd) and dense.stride(1) == 1
     _check(f(q_in.data_ptr(), q_in.stride(0), kv_in.data_ptr(), kv_in.stride(0), _ptr(g_in),
@@ -900,31 +901,34 @@ def latent_prepare(q_in, kv_in, g_in, norm_w, eps, inv_freq, rot, q_scale, q_nop
              q_nope.data_ptr(), q_nope.stride(0), q_lat.data_ptr(), q_lat.stride(0), _ptr(gate), _ptr(cache),
              dtype_code(q_lat.dtype), _ptr(page_table), page_table.shape[1] if page_table is not None else 1, page_size,
              tok_pos.data_ptr(), tok_seq.data_ptr(), seq_slot.data_ptr(), t, heads, dim, rd, rank, _ptr(dense),
-             dense.stride(0) if dense is not None else 0, 1 if half_layout else 0, _stream()),
+             dense.stride(0) if dense is not None else 0, 1 if half_layout else 0, float(rot_magnitude), _stream()),
            "latent_prepare", "elementwise", _nbytes(q_in, kv_in, q_nope) + t * (rank + 2 * rd) * q_lat.element_size())
 
 
-def heads_gemm(x, w, y, heads, scale=None):
+def heads_gemm(x, w, y, heads, scale=None, gate=None):
     """y[t, h, :] = scale[t, h] * w[h] @ x[t, h, :] for every head: x [T, heads, K] and y [T, heads, N]
     as views of 2-D tensors (the head stride may be wider than K or N), w [heads, N, K] contiguous,
-    scale float32 [T, heads] or None.  Float32 accumulation in ascending k."""
-    _cuda(x, w, y, scale)
+    scale float32 [T, heads] or None; ``gate`` float32 [T, heads * N] (rows may be wider) or None: the
+    results times sigmoid(gate).  Float32 accumulation in ascending k."""
+    _cuda(x, w, y, scale, gate)
     t, _, k = x.shape
     n = w.shape[1]
     assert x.shape[1] == heads and w.shape == (heads, n, k) and y.shape == (t, heads, n) and w.is_contiguous()
     assert x.stride(2) == 1 and y.stride(2) == 1 and x.dtype == w.dtype == y.dtype
     if scale is not None:
         assert scale.dtype == torch.float32 and scale.shape == (t, heads) and scale.is_contiguous()
+    if gate is not None:
+        assert gate.dtype == torch.float32 and gate.shape == (t, heads * n) and gate.stride(1) == 1
     if (x.dtype == torch.bfloat16 and k % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0
             and x.data_ptr() % 16 == 0 and t >= HEADS_GEMM_TC_MIN_TOKENS):
         grouped_gemm(x, x.stride(0), x.stride(1), None, 1, w, n * k, y, y.stride(0), y.stride(1), scale, None, heads, 1,
-                     None, heads, t, t, n, k, what="heads_gemm_tc", nbytes=_nbytes(w) + t * heads * (n + k) * 2)
+                     None, heads, t, t, n, k, gate=gate, gate_gstride=n, what="heads_gemm_tc", nbytes=_nbytes(w) + t * heads * (n + k) * 2)
         return
     f = _fn("latent_attention", "gb_heads_gemm",
             [c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_int, c_int,
-             c_int, c_int, c_void_p])
+             c_int, c_int, c_void_p, c_longlong, c_void_p])
     _check(f(x.data_ptr(), x.stride(0), x.stride(1), w.data_ptr(), y.data_ptr(), y.stride(0), y.stride(1), _ptr(scale),
-             dtype_code(x.dtype), t, heads, n, k, _stream()), "heads_gemm", "matmul",
+             dtype_code(x.dtype), t, heads, n, k, _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()), "heads_gemm", "matmul",
            _nbytes(w) + t * heads * (n + k) * x.element_size())
 
 
@@ -936,21 +940,25 @@ HEADS_GEMM_TC_MIN_TOKENS = 1
 
 def grouped_gemm(a, lda, a_gstride, a_rows, a_div, w, w_gstride, c, ldc, c_gstride, scale, scale_rows, s_rstride, s_gstride,
                  offsets, groups, rows, max_rows, n, k, gated=False, limit=0.0, alpha=0.0, shift=0.0, what="grouped_gemm",
-                 nbytes=0):
+                 nbytes=0, gate=None, gate_gstride=0, scale_in=False):
     """Many bfloat16 products C_g = A_g W_g^T of unequal row counts in one tensor-core launch (see
     csrc/grouped_gemm.cu): group g's rows are offsets[g]..offsets[g+1] (None: ``rows`` each), an A
     row is a_rows[i] // a_div (None: i), C is bfloat16 or float32 by its dtype; ``gated``: W_g stacks
     gate rows over up rows and C = min(g, limit) * sigmoid(alpha g) * (clamp(u) + shift); ``gated`` 2 / 3:
-    no gate rows, C = gelu(A W_g^T) in the exact (erf) form / relu(A W_g^T)^2."""
-    _cuda(a, w, c, scale, scale_rows, offsets, a_rows)
+    no gate rows, C = gelu(A W_g^T) in the exact (erf) form / relu(A W_g^T)^2.  ``gate`` (float32, not
+    with ``gated``): C times sigmoid(gate[row, g * gate_gstride + column]).  ``scale_in`` (with ``gated``):
+    the scale multiplies both sums before the activation instead of the result."""
+    _cuda(a, w, c, scale, scale_rows, offsets, a_rows, gate)
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
     assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and c.dtype in (torch.bfloat16, torch.float32)
     f = _fn("grouped_gemm", "gb_grouped_gemm",
             [c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_longlong,
              c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-             c_float, c_float, c_void_p])
+             c_float, c_float, c_void_p, c_longlong, c_longlong, c_int, c_void_p])
     _check(f(a.data_ptr(), lda, a_gstride, _ptr(a_rows), a_div, w.data_ptr(), w_gstride, c.data_ptr(), ldc, c_gstride,
              _ptr(scale), _ptr(scale_rows), s_rstride, s_gstride, _ptr(offsets), groups, rows, max_rows, n, k,
-             int(gated), 1 if c.dtype == torch.float32 else 0, limit, alpha, shift, _stream()), what, "matmul", nbytes)
+             int(gated), 1 if c.dtype == torch.float32 else 0, limit, alpha, shift, _ptr(gate),
+             gate.stride(0) if gate is not None else 0, gate_gstride, 1 if scale_in else 0, _stream()), what, "matmul", nbytes)
 
 
 def latent_attention_ref(qa, out, heads, rank, rd, cache, page_table, page_size, tok_pos, tok_seq, seq_slot, window=None,
@@ -970,16 +978,16 @@ def latent_attention_ref(qa, out, heads, rank, rd, cache, page_table, page_size,
            "attention", _nbytes(qa, out) + cache_bytes)
 
 
-def rope_pairs(x, tok_pos, inv_freq, rot):
+def rope_pairs(x, tok_pos, inv_freq, rot, magnitude: float = 1.0):
     """Rotates, in place, the first ``rot`` dims of every head of x [T, heads, hd] as interleaved
-    pairs (2i, 2i + 1) by the angle float32(position) * inv_freq[i]."""
+    pairs (2i, 2i + 1) by the angle float32(position) * inv_freq[i], cosines and sines times ``magnitude``."""
     _cuda(x, tok_pos, inv_freq)
     t, heads, hd = x.shape
     assert x.stride(2) == 1 and x.stride(1) == hd and inv_freq.dtype == torch.float32 and inv_freq.numel() == rot // 2
     f = _fn("latent_attention", "gb_rope_pairs", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-                                                  c_int, c_void_p])
+                                                  c_int, c_float, c_void_p])
     _check(f(x.data_ptr(), x.stride(0), dtype_code(x.dtype), tok_pos.data_ptr(), inv_freq.data_ptr(), t, heads, hd, rot,
-             _stream()), "rope_pairs", "elementwise", 2 * t * heads * rot * x.element_size())
+             float(magnitude), _stream()), "rope_pairs", "elementwise", 2 * t * heads * rot * x.element_size())
 
 
 def latent_attention_mma_usable(dtype, rank: int, rd: int, page_size: int) -> bool:
@@ -996,14 +1004,15 @@ _latent_scratch = {}
 
 def latent_attention_mma(qa, out, heads, rank, rd, cache, page_table, page_size, cu_seqlens, seq_start, seq_slot,
                          max_new: int, window=None, ksplits: int = 1, cache_bytes: int = 0, head_stride: int = 0,
-                         out_scale=None):
+                         out_scale=None, out_gate=None):
     """bfloat16 latent attention on the tensor cores (mma.sync) for packed sequences that bring any
     number of tokens each; with ``ksplits`` > 1 the keys of a tile of rows are dealt to that many
     CTAs and a second kernel adds their parts.  ``head_stride`` > 0: every head has rows of its own,
     ``cache`` [heads, packed tokens + 64, rank + rd] (elements ``head_stride`` apart), a sequence's rows
     from its first packed token on, every sequence from position 0, no page table; ``out_scale``
-    float32 [T, heads] multiplies the output."""
-    _cuda(qa, out, cache, page_table, cu_seqlens, seq_start, seq_slot, out_scale)
+    float32 [T, heads] multiplies the output, sigmoid(``out_gate``) too (float32 [T, heads * rank], rows may be wider)."""
+    _cuda(qa, out, cache, page_table, cu_seqlens, seq_start, seq_slot, out_scale, out_gate)
+    assert out_gate is None or (out_gate.dtype == torch.float32 and out_gate.shape[1] == heads * rank and out_gate.stride(1) == 1)
     if not latent_attention_mma_usable(qa.dtype, rank, rd, page_size):
         raise KernelError(f"latent_attention_mma: latent {rank} + {rd}, pages of {page_size} or {qa.dtype} not supported")
     assert qa.stride(-1) == 1 and out.stride(-1) == 1 and out.dtype == cache.dtype == torch.bfloat16 and cache.is_contiguous()
@@ -1022,11 +1031,13 @@ def latent_attention_mma(qa, out, heads, rank, rd, cache, page_table, page_size,
             part = _latent_scratch[qa.device.index] = torch.empty(max(need, 1 << 20), dtype=torch.float32, device=qa.device)
     f = _fn("latent_attention_mma", "gb_latent_attention_mma",
             [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
-             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_longlong, c_void_p, c_void_p], defines=defines)
+             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_longlong, c_void_p, c_void_p, c_longlong,
+             c_void_p], defines=defines)
     _check(f(qa.data_ptr(), qa.stride(0), out.data_ptr(), out.stride(0), _ptr(part), cache.data_ptr(), _ptr(page_table),
              page_table.shape[1] if page_table is not None else 1, page_size, cu_seqlens.data_ptr(), seq_start.data_ptr(),
              seq_slot.data_ptr(), seq_slot.numel(), ntok, heads, rank, rd, max_new * (1 if head_stride else heads),
-             window or 0, ksplits, head_stride, _ptr(out_scale), _stream()),
+             window or 0, ksplits, head_stride, _ptr(out_scale), _ptr(out_gate), out_gate.stride(0) if out_gate is not None else 0,
+             _stream()),
            "latent_attention_mma", "attention", _nbytes(qa, out) + cache_bytes)
     if ksplits > 1:
         count_launches(1)   # the merge kernel
@@ -1082,7 +1093,7 @@ def latent_attention_units(compute: str, rank: int, rd: int, dim: int = 0, vd: i
 
 # --------------------------------------------------------------------------- routed feed-forward
 
-ROUTINGS = {"softmax_top": 0, "softmax_all": 1, "sigmoid": 2}
+ROUTINGS = {"softmax_top": 0, "softmax_all": 1, "sigmoid": 2, "sigmoid_raw": 3}
 
 
 def moe_topk(z, bias, experts, top, has_gate=False, routing="softmax_top", scale: float = 1.0):
@@ -1090,8 +1101,8 @@ def moe_topk(z, bias, experts, top, has_gate=False, routing="softmax_top", scale
     logits z (float32 [T, experts (+ 1)]): each token's ``top`` largest z + bias (the lower index wins
     a tie), weighed by ``routing`` times ``scale``: "softmax_top" the softmax over those alone,
     "softmax_all" their shares of the softmax over all experts, which do not add up to one; "sigmoid":
-    scores s = sigmoid(z), the ``top`` largest s + bias, each s over the sum of the chosen s (+ 1e-20).
-    With ``has_gate`` the sigmoid of column ``experts``."""
+    scores s = sigmoid(z), the ``top`` largest s + bias, each s over the sum of the chosen s (+ 1e-20);
+    "sigmoid_raw" the same choice, each s as it is.  With ``has_gate`` the sigmoid of column ``experts``."""
     _cuda(z, bias)
     t = z.shape[0]
     assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape[1] >= experts + (1 if has_gate else 0)
@@ -1107,11 +1118,12 @@ def moe_topk(z, bias, experts, top, has_gate=False, routing="softmax_top", scale
 
 
 def moe_experts(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down, residual, limit, shared_limit, alpha,
-                shift, col_scale=None):
+                shift, col_scale=None, weigh_input=False, store=False):
     """residual[t] += sum_k wts[t, k] * expert_{idx[t, k]}(h[t]) + sg[t] * shared(h[t]), token-major
     (two kernels: gate/up with the activation, then down).  w_gate_up [E, 2 ff, width] (gate rows,
     then up rows), w_down [E, width, ff]; the shared expert's [2 ffs, width] and [width, ffs], or None.
-    ``col_scale`` (float32 [width]) multiplies what is added."""
+    ``col_scale`` (float32 [width]) multiplies what is added.  ``weigh_input``: the weights multiply the
+    experts' inputs, expert(wts[t, k] * h[t]).  ``store``: the result replaces the rows of ``residual``."""
     _check_col_scale(col_scale, h.shape[1])
     _cuda(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down, residual)
     t, width = h.shape
@@ -1127,24 +1139,26 @@ def moe_experts(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down,
     slots = top + (1 if shared_down is not None else 0)
     y = torch.empty((t, slots, max(ff, ffs)), dtype=h.dtype, device=h.device)
     f = _fn("moe", "gb_moe_gate_up", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                      c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_void_p])
+                                      c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_void_p, c_void_p])
     _check(f(h.data_ptr(), h.stride(0), dtype_code(h.dtype), idx.data_ptr(), w_gate_up.data_ptr(), _ptr(shared_gate_up),
-             y.data_ptr(), t, width, ff, ffs, top, limit, shared_limit, alpha, shift, _stream()), "moe_gate_up", "matmul",
+             y.data_ptr(), t, width, ff, ffs, top, limit, shared_limit, alpha, shift, wts.data_ptr() if weigh_input else None,
+             _stream()), "moe_gate_up", "matmul",
            _nbytes(h, y) + t * slots * 2 * ff * width * h.element_size())
     rows = torch.empty((t, slots, width), dtype=torch.float32, device=h.device)
     f = _fn("moe", "gb_moe_down", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                   c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
-    _check(f(y.data_ptr(), dtype_code(h.dtype), idx.data_ptr(), wts.data_ptr(), _ptr(sg), w_down.data_ptr(),
-             _ptr(shared_down), rows.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, ff, ffs, top,
-             _ptr(col_scale), _stream()),
+                                   c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p])
+    _check(f(y.data_ptr(), dtype_code(h.dtype), idx.data_ptr(), None if weigh_input else wts.data_ptr(), _ptr(sg),
+             w_down.data_ptr(), _ptr(shared_down), rows.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, ff, ffs,
+             top, _ptr(col_scale), 1 if store else 0, _stream()),
            "moe_down", "matmul", _nbytes(y) + 2 * _nbytes(rows) + 2 * t * width * 4 + t * slots * ff * width * h.element_size())
     count_launches(1)   # the kernel that adds a token's rows
 
 
-def moe_experts_plain(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None):
+def moe_experts_plain(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None, store=False):
     """residual[t] += sum_k wts[t, k] * down_{idx[t, k]} act(up_{idx[t, k]} h[t]) for experts without a
     gate (``act`` one of PLAIN_ACTS), token-major.  w_up [E, ff, width], w_down [E, width, ff].
-    ``col_scale`` (float32 [width]) multiplies what is added."""
+    ``col_scale`` (float32 [width]) multiplies what is added.  ``store``: the result replaces the rows of
+    ``residual``."""
     _check_col_scale(col_scale, h.shape[1])
     _cuda(h, idx, wts, w_up, w_down, residual)
     t, width = h.shape
@@ -1158,15 +1172,15 @@ def moe_experts_plain(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale
              PLAIN_ACTS[act], _stream()), "moe_up", "matmul", _nbytes(h, y) + t * top * ff * width * h.element_size())
     rows = torch.empty((t, top, width), dtype=torch.float32, device=h.device)
     f = _fn("moe", "gb_moe_down", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                   c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+                                   c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p])
     _check(f(y.data_ptr(), dtype_code(h.dtype), idx.data_ptr(), wts.data_ptr(), None, w_down.data_ptr(), None,
              rows.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, ff, 0, top, _ptr(col_scale),
-             _stream()),
+             1 if store else 0, _stream()),
            "moe_down", "matmul", _nbytes(y) + 2 * _nbytes(rows) + 2 * t * width * 4 + t * top * ff * width * h.element_size())
     count_launches(1)   # the kernel that adds a token's rows
 
 
-def moe_experts_plain_grouped(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None):
+def moe_experts_plain_grouped(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None, store=False):
     """As moe_experts_plain for a step of many tokens: entries ordered by expert, two grouped
     tensor-core products (up with the activation in its epilogue, down scaled by the routing weights), a
     token's rows added into the residual in slot order."""
@@ -1188,13 +1202,14 @@ def moe_experts_plain_grouped(h, idx, wts, w_up, w_down, residual, act="gelu", c
     grouped_gemm(y, ff, 0, None, 1, w_down, width * ff, rows, width, 0, wts.view(-1), perm, 1, 0, offsets, e, 0, entries,
                  width, ff, what="moe_down_tc", nbytes=_nbytes(w_down, y, rows))
     _check_col_scale(col_scale, width)
-    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_int,
+                                                c_void_p])
     _check(f(rows.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _ptr(col_scale),
-             _stream()),
+             1 if store else 0, _stream()),
            "moe_combine", "elementwise", _nbytes(rows) + 2 * t * width * 4)
 
 
-def moe_experts_plain_tc(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None):
+def moe_experts_plain_tc(h, idx, wts, w_up, w_down, residual, act="gelu", col_scale=None, store=False):
     """As moe_experts_plain_grouped for a prompt step, the two products on the tcgen05 kernel (the
     activations copied into an order in which every expert's rows start at a multiple of the
     tile's tokens; the activation and the routing weight in the first product's epilogue)."""
@@ -1220,9 +1235,10 @@ def moe_experts_plain_tc(h, idx, wts, w_up, w_down, residual, act="gelu", col_sc
     out = torch.empty((rows, width), dtype=torch.float32, device=h.device)
     gemm_tc_grouped(y, w_down.view(e * width, ff), out, width, e, tile_expert)
     _check_col_scale(col_scale, width)
-    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_int,
+                                                c_void_p])
     _check(f(out.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _ptr(col_scale),
-             _stream()),
+             1 if store else 0, _stream()),
            "moe_combine", "elementwise", entries * width * 4 + 2 * t * width * 4)
 
 
@@ -1237,7 +1253,7 @@ def moe_grouped_usable(h, w_gate_up, w_down) -> bool:
 
 
 def moe_experts_grouped(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down, residual, limit, shared_limit,
-                        alpha, shift, col_scale=None):
+                        alpha, shift, col_scale=None, weigh_input=False, store=False):
     """As moe_experts for a step of many tokens: the (token, slot) entries are ordered by expert on the
     device, each expert's rows run as one product of a grouped tensor-core launch (gate/up with the
     activation, then down scaled by the routing weights), a token's rows are added into the residual
@@ -1254,16 +1270,19 @@ def moe_experts_grouped(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shar
     _check(f(idx.data_ptr(), entries, e, offsets.data_ptr(), perm.data_ptr(), place.data_ptr(), _stream()), "moe_sort",
            "elementwise", 3 * entries * 4)
     y = torch.empty((entries, ff), dtype=torch.bfloat16, device=h.device)
-    grouped_gemm(h, h.stride(0), 0, perm, top, w_gate_up, ff2 * width, y, ff, 0, None, None, 0, 0, offsets, e, 0, entries,
-                 ff, width, gated=True, limit=limit, alpha=alpha, shift=shift, what="moe_gate_up_tc",
-                 nbytes=_nbytes(w_gate_up, y) + entries * width * 2)
+    weights = (wts.view(-1), perm, 1)                    # an entry's weight: on its input, or on its result
+    none = (None, None, 0)
+    grouped_gemm(h, h.stride(0), 0, perm, top, w_gate_up, ff2 * width, y, ff, 0, *(weights if weigh_input else none), 0, offsets,
+                 e, 0, entries, ff, width, gated=True, limit=limit, alpha=alpha, shift=shift, scale_in=weigh_input,
+                 what="moe_gate_up_tc", nbytes=_nbytes(w_gate_up, y) + entries * width * 2)
     rows = torch.empty((entries, width), dtype=torch.float32, device=h.device)
-    grouped_gemm(y, ff, 0, None, 1, w_down, width * ff, rows, width, 0, wts.view(-1), perm, 1, 0, offsets, e, 0, entries,
-                 width, ff, what="moe_down_tc", nbytes=_nbytes(w_down, y, rows))
+    grouped_gemm(y, ff, 0, None, 1, w_down, width * ff, rows, width, 0, *(none if weigh_input else weights), 0, offsets, e, 0,
+                 entries, width, ff, what="moe_down_tc", nbytes=_nbytes(w_down, y, rows))
     _check_col_scale(col_scale, width)
-    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_int,
+                                                c_void_p])
     _check(f(rows.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _ptr(col_scale),
-             _stream()),
+             1 if store else 0, _stream()),
            "moe_combine", "elementwise", _nbytes(rows) + 2 * t * width * 4)
     _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, alpha, shift, col_scale)
 
@@ -1280,12 +1299,13 @@ def moe_tc_usable(h, w_gate_up, w_down) -> bool:
 
 
 def gemm_tc_grouped(x, w, y, n, experts, tile_expert, row_scale=None, gated=False, limit=0.0, alpha=0.0, shift=0.0,
-                    bn=MOE_TC_TILE, act=None):
+                    bn=MOE_TC_TILE, act=None, scale_in=False):
     """The tcgen05 product over groups of rows: x [rows, K] holds the groups one after the other, each
     starting at a multiple of ``bn`` rows; w stacks the groups' matrices ([experts * n, K], or
     [experts * 2 n, K] gated); tile_expert names the group of every tile of ``bn`` rows (-1: none).
     y float32 [rows, n], or with ``gated`` bfloat16 [rows, n] = row_scale * act(gate, up), or with
-    ``act`` (one of PLAIN_ACTS) bfloat16 [rows, n] = row_scale * act(x w^T) (no gate rows)."""
+    ``act`` (one of PLAIN_ACTS) bfloat16 [rows, n] = row_scale * act(x w^T) (no gate rows).  ``scale_in``
+    (gated): act(row_scale * gate, row_scale * up)."""
     _cuda(x, w, y, tile_expert, row_scale)
     rows, k = x.shape
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.stride(1) == 1 and w.is_contiguous()
@@ -1294,15 +1314,15 @@ def gemm_tc_grouped(x, w, y, n, experts, tile_expert, row_scale=None, gated=Fals
     assert tile_expert.dtype == torch.int32 and tile_expert.numel() == rows // bn and rows % bn == 0
     f = _fn("gemm_tc", "gb_gemm_tc_grouped",
             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_int, c_int, c_int, c_void_p,
-             c_void_p, c_float, c_float, c_float, c_int, c_void_p])
+             c_void_p, c_float, c_float, c_float, c_int, c_int, c_void_p])
     _check(f(x.data_ptr(), w.data_ptr(), y.data_ptr(), 3 if gated else (0 if act else 1), rows, n, k, x.stride(0), y.stride(0), bn,
              sm_count(x.device), experts, tile_expert.data_ptr(), _ptr(row_scale), limit, alpha, shift, PLAIN_ACTS[act],
-             _stream()),
+             1 if scale_in else 0, _stream()),
            "gemm_tc_grouped", "matmul", _nbytes(x, w, y))
 
 
 def moe_experts_tc(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_down, residual, limit, shared_limit, alpha,
-                   shift, col_scale=None):
+                   shift, col_scale=None, weigh_input=False, store=False):
     """As moe_experts_grouped for a prompt step, the experts' two products on the tcgen05 kernel: the
     activations are copied into an order in which every expert's rows start at a multiple of the
     tile's tokens (zeros between), the routing weight multiplies the activation's rows, and a token's
@@ -1326,13 +1346,14 @@ def moe_experts_tc(h, idx, wts, sg, w_gate_up, w_down, shared_gate_up, shared_do
              scale.data_ptr(), rows, width, top, bn, _stream()), "moe_permute", "elementwise", 2 * entries * width * 2)
     y = torch.empty((rows, ff), dtype=torch.bfloat16, device=h.device)
     gemm_tc_grouped(xp, w_gate_up.view(e * ff2, width), y, ff, e, tile_expert, scale, gated=True, limit=limit, alpha=alpha,
-                    shift=shift)
+                    shift=shift, scale_in=weigh_input)
     out = torch.empty((rows, width), dtype=torch.float32, device=h.device)
     gemm_tc_grouped(y, w_down.view(e * width, ff), out, width, e, tile_expert)
     _check_col_scale(col_scale, width)
-    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
+    f = _fn("grouped_gemm", "gb_moe_combine", [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_int,
+                                                c_void_p])
     _check(f(out.data_ptr(), place.data_ptr(), residual.data_ptr(), residual.stride(0), t, width, top, _ptr(col_scale),
-             _stream()),
+             1 if store else 0, _stream()),
            "moe_combine", "elementwise", entries * width * 4 + 2 * t * width * 4)
     _shared_expert(h, sg, shared_gate_up, shared_down, residual, shared_limit, alpha, shift, col_scale)
 
@@ -1869,12 +1890,15 @@ def matrix_memory(q, k, v, in_logit, forget_logit, state, aux, cu_seqlens, seq_s
 
 def filter_rope_cache(u, taps, state, inv_freq, rot, ctx_pos, tok_seq, seq_slot, cu_seqlens, page_table, page_size, q_out,
                       kcache, vcache, heads, groups, dim, vdim, q_norm=None, k_norm=None, norm_eps: float = 0.0,
-                      rot_magnitude: float = 1.0, q_temper=None, values_are_keys: bool = False):
+                      rot_magnitude: float = 1.0, q_temper=None, values_are_keys: bool = False, pairs: bool = False,
+                      unit_after: bool = False):
     """The columns [q | k | v] of ``u`` through a short causal filter (``taps`` [channels, K] or
-    None), the first ``rot`` dims of each q and k head rotated (pairs i, i + rot/2), then q into
+    None), the first ``rot`` dims of each q and k head rotated (pairs i, i + rot/2, or with ``pairs`` 2i,
+    2i + 1), then q into
     ``q_out`` [T, heads * dim] and keys and values into their pages (None: not kept).
     ``q_norm`` / ``k_norm`` (float32 [dim]): every q / k head is divided by its root mean square
-    (``norm_eps``) and multiplied by the weight before the rotation.  ``rot_magnitude`` multiplies
+    (``norm_eps``) and multiplied by the weight before the rotation; ``unit_after`` (instead): divided by
+    it after the rotation, without a weight.  ``rot_magnitude`` multiplies
     the cosines and sines.  ``q_temper`` (coef, every): q at position p times 1 + coef ln(floor((p +
     1) / every) + 1).  ``values_are_keys``: the rows hold [q | k] alone and a value head is its key
     head as projected and filtered, before norm and rotation (vdim == dim)."""
@@ -1898,12 +1922,12 @@ def filter_rope_cache(u, taps, state, inv_freq, rot, ctx_pos, tok_seq, seq_slot,
     f = _fn("attention_capped", "gb_filter_rope_cache_ext",
             [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
              c_void_p, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
-             c_void_p, c_float, c_float, c_float, c_int, c_int, c_void_p])
+             c_void_p, c_float, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p])
     _check(f(up, dtype_code(u.dtype), ldu, _ptr(taps), _ptr(state) if k > 1 else None, k, _ptr(inv_freq) if rot else None,
              rot, ctx_pos.data_ptr(), tok_seq.data_ptr(), seq_slot.data_ptr(), cu_seqlens.data_ptr(), _ptr(page_table),
              page_table.shape[1] if page_table is not None else 1, page_size, qp, ldq, _ptr(kcache), _ptr(vcache),
              u.shape[0], heads, groups, dim, vdim, _ptr(q_norm), _ptr(k_norm), float(norm_eps), float(rot_magnitude), qt_coef,
-             qt_every, 1 if values_are_keys else 0, _stream()), "filter_rope_cache", "elementwise",
+             qt_every, 1 if values_are_keys else 0, 1 if pairs else 0, 1 if unit_after else 0, _stream()), "filter_rope_cache", "elementwise",
            2 * u.numel() * u.element_size())
 
 

@@ -28,6 +28,9 @@ Interfaces (all tensors on the device; ``ctx`` is the ``StepContext`` of the run
   needs in the order of ``parts()`` (``Block.split_caches`` deals them out).
 * scale: ``factor()`` -> float32 [hidden], a factor per feature on what a mixer or feed-forward adds; the
   block hands it to the part's ``set_output_scale`` once both are loaded.
+  A mixer or feed-forward with ``set_output_store()`` can be asked, before it is loaded, to store its output
+  into the rows it is given instead of adding it (a block that hands it rows of its own); ``stores`` then
+  says whether it does.
 * stream: ``forward(ctx, x, then_norm=None)`` changes the residual stream between two runs of layers
   (``ScheduleEntry.before``) and returns ``then_norm``'s output when it made it in the same pass.
 * embedding: ``forward(ctx, tokens, out)``; head: ``forward(ctx, h)`` -> float32 logits.

@@ -174,8 +174,10 @@ class ParallelBlock(Block):
 
 class SandwichBlock(Block):
     """``sandwich``: x += mixer_post_norm(mixer(mixer_norm(x))); x += ffn_post_norm(ffn(ffn_norm(x))).
-    A sublayer adds its output into float32 rows of zeros instead of the residual stream; the norm
-    after it reads those rows and adds the normed rows into the stream.  The layer's spec lists
+    A sublayer's output goes into float32 rows of its own instead of the residual stream (stored there by
+    parts that can, else added into zeros); the norm after it reads those rows, adds the normed rows into
+    the stream and makes the output of the norm that reads the stream next, the next layer's first one
+    included, in the same pass.  The layer's spec lists
     ``mixer_norm``, ``mixer``, ``mixer_post_norm`` and, when the layer has a feed-forward,
     ``ffn_norm``, ``ffn``, ``ffn_post_norm``."""
 
@@ -187,6 +189,9 @@ class SandwichBlock(Block):
         self.ffn = self.need("ffn", "ffn") if "ffn" in layer_spec.parts else None
         self.ffn_norm = self.need("ffn_norm", "norm") if self.ffn is not None else None
         self.ffn_post_norm = self.need("ffn_post_norm", "norm") if self.ffn is not None else None
+        for part in (self.mixer, self.ffn):
+            if hasattr(part, "set_output_store"):
+                part.set_output_store()
 
     def parts(self):
         out = {"mixer_norm": self.mixer_norm, "mixer": self.mixer, "mixer_post_norm": self.mixer_post_norm}
@@ -194,21 +199,41 @@ class SandwichBlock(Block):
             out.update({"ffn_norm": self.ffn_norm, "ffn": self.ffn, "ffn_post_norm": self.ffn_post_norm})
         return out
 
-    def forward(self, ctx, x, caches, writes_cache=True):
+    #: forward takes ``h_in`` / ``next_norm``: the norm before may be made by the pass of the norm after
+    chains_norms = True
+    takes_unscaled_rows = True
+
+    def first_norm(self):
+        return self.mixer_norm
+
+    @staticmethod
+    def _rows_for(part, x):
+        """Float32 rows for the part's output: as they come for a part that stores, else zeros."""
+        return torch.empty_like(x) if _stores(part) else torch.zeros_like(x)
+
+    def forward(self, ctx, x, caches, writes_cache=True, h_in=None, next_norm=None):
         mine = self.split_caches(caches)
-        y = torch.zeros_like(x)
-        self.mixer.forward(ctx, self.mixer_norm.forward(ctx, x), y, mine["mixer"], writes_cache)
+        y = self._rows_for(self.mixer, x)
+        self.mixer.forward(ctx, _plain(h_in) if h_in is not None else self.mixer_norm.forward(ctx, x), y, mine["mixer"], writes_cache)
         if self.ffn is None:
-            self.mixer_post_norm.add_normed(ctx, y, x)
-            return
-        # the norm after the mixer and the norm before the feed-forward read the same rows: one pass
-        fused = isinstance(self.ffn_norm, type(self.mixer_post_norm)) and hasattr(self.ffn_norm, "weight")
-        h = self.mixer_post_norm.add_normed(ctx, y, x, self.ffn_norm if fused else None)
+            return self.mixer_post_norm.add_normed(ctx, y, x, _same_kind(self.mixer_post_norm, next_norm))
+        h = self.mixer_post_norm.add_normed(ctx, y, x, _same_kind(self.mixer_post_norm, self.ffn_norm))
         if h is None:
             h = self.ffn_norm.forward(ctx, x)
-        y.zero_()
+        if not _stores(self.ffn):
+            y.zero_()
         self.ffn.forward(ctx, h, y)
-        self.ffn_post_norm.add_normed(ctx, y, x)
+        return self.ffn_post_norm.add_normed(ctx, y, x, _same_kind(self.ffn_post_norm, next_norm))
+
+
+def _stores(part):
+    """Whether the part stores its output instead of adding it (it was asked to, and could)."""
+    return getattr(part, "stores", False)
+
+
+def _same_kind(norm, then):
+    """``then`` if ``norm``'s pass over a sublayer's output can make its output as well, else None."""
+    return then if isinstance(then, type(norm)) and hasattr(then, "weight") else None
 
 
 def _plain(h):

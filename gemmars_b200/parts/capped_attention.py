@@ -4,7 +4,7 @@ wider or narrower than their keys, or whose q, k and v pass a short filter over 
 For one token, with h the mixer's input:
   q, k, v = W_q h, W_k h, W_v h (+ biases), heads x dim, kv_heads x dim, kv_heads x vdim;
   each channel passes a causal filter over time (``conv`` taps, no bias, no activation; 0: none);
-  the position encoding turns q and k (a ``rotary`` part with the "half" layout, or None);
+  the position encoding turns q and k (a ``rotary`` part of either layout, or None);
   score = (q . k) * scale, then cap * tanh(score / cap) when ``softcap``; a query sees itself and
   the ``window`` - 1 positions before it (None: all), and with ``keep_first`` the sequence's first
   ``keep_first`` positions as well, at their true places, however far the window has moved on;
@@ -27,9 +27,10 @@ its dims (``q_norm``, ``k_norm``, shared by the heads) before the rotation.  ``q
 "every"}: the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
 ``fixed_sink`` (a number s): exp(s) joins the softmax's denominator for every head, without a
 tensor (0.0: one is added to the denominator).  ``gate`` may be "head": one number per head,
-sigmoid(W_g h)[head], instead of one per output channel.
+sigmoid(W_g h)[head], instead of one per output channel.  ``qk_unit`` (an eps; default none): every q
+and k head is divided by its root mean square over its dims after the rotation, without a weight.
 Parameters: hidden_size, heads, kv_heads, dim, vdim, bias, conv, window, keep_first, sink, scale,
-softcap, gate, position, has_kv, ring, out_scale, values_are_keys, qk_norm, q_temper, fixed_sink.
+softcap, gate, position, has_kv, ring, out_scale, values_are_keys, qk_norm, qk_unit, q_temper, fixed_sink.
 """
 from __future__ import annotations
 
@@ -66,6 +67,9 @@ class CappedAttention(Part):
         self.out_scale = float(p.get("out_scale", 1.0))
         self.values_are_keys = bool(p.get("values_are_keys", False))
         self.qk_norm_eps = float(p["qk_norm"]) if p.get("qk_norm") is not None else None
+        self.qk_unit_eps = float(p["qk_unit"]) if p.get("qk_unit") is not None else None
+        if self.qk_norm_eps is not None and self.qk_unit_eps is not None:
+            raise ValueError("capped_attention: a norm of q and k before the rotation and one after it exclude each other")
         temper = p.get("q_temper")
         self.q_temper = (float(temper["coef"]), int(temper["every"])) if temper else None
         self.fixed_sink = float(p["fixed_sink"]) if p.get("fixed_sink") is not None else None
@@ -90,11 +94,12 @@ class CappedAttention(Part):
             raise ValueError(f"capped_attention: keep_first must not be negative, got {self.keep_first}")
         pos = p.get("position")
         self.position = build_part("position", pos, compute) if pos is not None else None
-        if self.position is not None and not (isinstance(self.position, Rotary) and self.position.layout == "half"):
-            raise ValueError("capped_attention: the position encoding must be a rotary part with the half layout")
+        if self.position is not None and not isinstance(self.position, Rotary):
+            raise ValueError("capped_attention: the position encoding must be a rotary part")
         self.own_kv = self.kv_heads if self.has_kv else 0
         own_v = 0 if self.values_are_keys else self.own_kv
         self.channels = (self.heads + self.own_kv) * self.dim + own_v * self.vdim     # q | k | v
+        self.stores = False
         self.proj = self.o = self.filter = self.sinks = self.q_norm = self.k_norm = None
 
     def wants(self):
@@ -131,6 +136,7 @@ class CappedAttention(Part):
             bias = torch.cat(parts)
         self.proj = Linear.stacked([t[n] for n in names], bias, 8 if self.gate_per_head else 1)   # one product: [q | k | v | gate]
         self.o = Linear(t["o"])
+        self.o.stores = self.stores
         if self.taps:
             self.filter = torch.cat([t[n + "_conv"] for n in qkv], dim=0).contiguous()
         if self.sink:
@@ -147,6 +153,10 @@ class CappedAttention(Part):
     def set_output_scale(self, scale):
         """``scale`` (float32 [hidden]) multiplies what the mixer adds."""
         self.o.out_scale = scale
+
+    def set_output_store(self):
+        """What the mixer would add is stored instead."""
+        self.stores = True
 
     def kernel_units(self):
         return (kernels.gemm_units(self.compute) + kernels.attention_capped_units(self.compute, self.dim, self.vdim)
@@ -183,9 +193,11 @@ class CappedAttention(Part):
         kernels.filter_rope_cache(p[:, :c], self.filter, filter_state, self.position.inv_freq(p.device) if rot else None, rot,
                                   ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, ctx.cu_seqlens, group.page_table, group.page_size,
                                   q, kc if self.has_kv else None, vc if self.has_kv else None, nh, self.own_kv, d, vd,
-                                  q_norm=self.q_norm, k_norm=self.k_norm, norm_eps=self.qk_norm_eps or 0.0,
+                                  q_norm=self.q_norm, k_norm=self.k_norm,
+                                  norm_eps=self.qk_norm_eps or self.qk_unit_eps or 0.0,
                                   rot_magnitude=self.position.magnitude if rot else 1.0, q_temper=self.q_temper,
-                                  values_are_keys=self.values_are_keys)
+                                  values_are_keys=self.values_are_keys, pairs=bool(rot) and self.position.layout == "interleaved",
+                                  unit_after=self.qk_unit_eps is not None)
         if self.taps > 1:
             kernels.short_filter_state(p[:, :c], filter_state, ctx.cu_seqlens, ctx.seq_slot, self.taps)
         att = torch.empty((t, nh * vd), dtype=p.dtype, device=p.device)

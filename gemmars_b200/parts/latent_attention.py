@@ -1,5 +1,5 @@
 """Latent attention: causal attention whose keys and values are expanded from one cached
-low-rank row per position, shared by all heads, with an optional sigmoid gate per head.
+low-rank row per position, shared by all heads, with an optional sigmoid gate per head or per number.
 
 For a token with input h at position p (H heads; per head ``dim`` unrotated and ``rot_dim``
 rotated query/key dims, value size ``vdim``; latent size ``rank``):
@@ -11,6 +11,8 @@ rotated query/key dims, value size ``vdim``; latent size ``rank``):
     s[h, j] = (q_nope[h] . Wuk[h] c_j + rotate(q_rot[h], p) . kr_j) * scale,  j <= p
     o[h]    = sigmoid(Wg h)[h] * sum_j softmax_j(s[h])[j] v_j[h];   residual += Wo concat(o)
 
+(with a ``window``, p - j < window as well).
+
 Only [c | kr] is cached, one row of ``rank + rot_dim`` values per position (a ``KVNeed`` with one
 kv head and no separate values).  Both expansions are moved off the keys: Wuk[h]^T is applied to
 the query (q_nope[h] . Wuk[h] c = (Wuk[h]^T q_nope[h]) . c) and Wuv[h] to the attention's output
@@ -20,9 +22,9 @@ single tokens all run one attention kernel over the cached rows, with all heads 
 With ``q_rank`` the queries pass a latent of their own: q = Wuq (rmsnorm(Wdq h) * w_q).
 
 All sizes and constants are parameters: hidden_size, num_heads, dim, rot_dim, vdim, rank, scale,
-norm_eps, gate (whether the output gate exists), window (None: all keys), q_rank (None: queries straight
-from h), position (a PartSpec of kind ``rotary``, of either layout, or None), out_scale (a factor on the
-result, applied in float32 after the output product).
+norm_eps, gate (True: one gate per head as above; "channel": one per output number, Wo (sigmoid(Wg h) *
+concat(o)); False: none), window (None: all keys), q_rank (None: queries straight from h), position (a PartSpec of kind ``rotary``, of either layout, with a magnitude or without, or None),
+out_scale (a factor on the result, applied in float32 after the output product).
 """
 from __future__ import annotations
 
@@ -49,13 +51,18 @@ class LatentAttention(Part):
         self.rank = int(p["rank"])
         self.scale = float(p["scale"])
         self.eps = float(p.get("norm_eps", 1e-6))
-        self.gated = bool(p.get("gate", True))
+        gate = p.get("gate", True)
+        if gate not in (True, False, None, "channel"):
+            raise ValueError(f"latent_attention: gate must be a truth value or 'channel', got {gate!r}")
+        self.gated = bool(gate)
+        self.gate_rows = 0 if not gate else (self.num_heads * self.vdim if gate == "channel" else self.num_heads)
+        self.gate_per_head = self.gated and gate != "channel"
         self.window = p.get("window")
         pos = p.get("position")
         self.position = build_part("position", pos, compute) if pos is not None else None
         if self.position is not None:
-            if not isinstance(self.position, Rotary) or self.position.magnitude != 1.0:
-                raise ValueError("latent_attention: the position encoding must be a rotary part without a magnitude, or none")
+            if not isinstance(self.position, Rotary):
+                raise ValueError("latent_attention: the position encoding must be a rotary part, or none")
             if self.position.rotary_dim > self.rot_dim:
                 raise ValueError(f"latent_attention: cannot rotate {self.position.rotary_dim} of {self.rot_dim} dims")
         if min(self.num_heads, self.rank, self.vdim) <= 0 or self.dim < 0 or self.rot_dim < 0 or self.dim + self.rot_dim <= 0:
@@ -64,6 +71,7 @@ class LatentAttention(Part):
         if self.q_rank is not None and self.q_rank < 1:
             raise ValueError(f"latent_attention: q_rank must be positive, got {self.q_rank}")
         self.out_scale = float(p.get("out_scale", 1.0))
+        self.stores = False
         self.proj = self.uq = self.o = self.uk_t = self.uv = self.norm_w = self.q_norm_w = None
 
     # ---- weights
@@ -79,7 +87,7 @@ class LatentAttention(Part):
                   "uk": TensorWant((nh * self.dim, r)), "uv": TensorWant((nh * self.vdim, r)),
                   "o": TensorWant((h, nh * self.vdim))})
         if self.gated:
-            w["g"] = TensorWant((nh, h))
+            w["g"] = TensorWant((self.gate_rows, h))
         return w
 
     def load(self, t):
@@ -87,11 +95,11 @@ class LatentAttention(Part):
         # one product reads the input once: queries (or their latent), then the latent and the key part,
         # then the gate logits
         first = t["q"] if self.q_rank is None else t["dq"]
-        self.proj = Linear.stacked([first, t["dkv"]] + ([t["g"]] if self.gated else []),
-                                   multiple=1 if self.q_rank is None else 4)
+        self.proj = Linear.stacked([first, t["dkv"]] + ([t["g"]] if self.gated else []), multiple=4)
         if self.q_rank is not None:
             self.uq, self.q_norm_w = Linear(t["uq"]), t["dq_norm"].contiguous()
         self.o = Linear(t["o"])
+        self.o.stores = self.stores
         if self.out_scale != 1.0:
             self.set_output_scale(None)
         # [heads, rank, dim]: the matrix that carries a head's unrotated query dims into the latent space
@@ -108,6 +116,10 @@ class LatentAttention(Part):
         if scale is None:
             scale = torch.ones(self.hidden_size, dtype=torch.float32, device=self.o.weight.device)
         self.o.out_scale = scale * self.out_scale
+
+    def set_output_store(self):
+        """What the mixer would add is stored instead."""
+        self.stores = self.out_scale == 1.0
 
     def kernel_units(self):
         units = kernels.gemm_units(self.compute) + kernels.latent_attention_units(self.compute, self.rank, self.rot_dim,
@@ -139,20 +151,25 @@ class LatentAttention(Part):
             q = self.uq(cq, out_dtype=torch.float32)
         q_nope = torch.empty((t, nh * dim), dtype=self.act_dtype, device=h.device)
         qa = torch.empty((t, nh * (r + rd)), dtype=self.act_dtype, device=h.device)
-        gate = torch.empty((t, nh), dtype=torch.float32, device=h.device) if self.gated else None
+        logits = proj[:, nq + r + rd:nq + r + rd + self.gate_rows] if self.gated else None
+        # one gate per head is made beside the queries and scales the heads' results; one per number is
+        # taken from its logits where the results are written
+        gate = torch.empty((t, nh), dtype=torch.float32, device=h.device) if self.gate_per_head else None
+        channel = logits if self.gated and not self.gate_per_head else None
         rot = self.position.rotary_dim if self.position is not None else 0
         # a prompt step whose sequences all start at position 0 (no cached prefix) may expand keys and
         # values per head, which is less arithmetic than attention over the latent rows
-        expand = (self.window is None and t >= kernels.LATENT_EXPAND_MIN_TOKENS and ctx.host is not None
+        expand = (t >= kernels.LATENT_EXPAND_MIN_TOKENS and ctx.host is not None
                   and not any(ctx.host["seq_start"]) and kernels.latent_expand_usable(h.dtype, r, dim, rd, vd))
         dense = torch.empty((t, r + rd), dtype=self.act_dtype, device=h.device) if expand else None
-        kernels.latent_prepare(q, proj[:, nq:nq + r + rd], proj[:, nq + r + rd:nq + r + rd + nh] if self.gated else None,
+        kernels.latent_prepare(q, proj[:, nq:nq + r + rd], logits if self.gate_per_head else None,
                                self.norm_w, self.eps, self.position.inv_freq(h.device) if rot else None, rot, self.scale,
                                q_nope, qa, gate, kc.view(-1, group.page_size, r + rd) if writes_cache else None,
                                group.page_table, group.page_size, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, nh, dim, rd, r,
-                               dense=dense, half_layout=self.position is not None and self.position.layout == "half")
+                               dense=dense, half_layout=self.position is not None and self.position.layout == "half",
+                               rot_magnitude=self.position.magnitude if rot else 1.0)
         if expand:
-            return self._expanded(ctx, q_nope, qa, gate, dense, residual)
+            return self._expanded(ctx, q_nope, qa, gate, channel, dense, residual)
         if dim:
             kernels.heads_gemm(q_nope.view(t, nh, dim), self.uk_t, qa.view(t, nh, r + rd)[:, :, :r], nh)
         else:
@@ -161,10 +178,10 @@ class LatentAttention(Part):
         kernels.latent_attention(ctx, qa, lat, nh, r, rd, kc.view(-1, group.page_size, r + rd), group.page_table,
                                  group.page_size, self.window)
         o = torch.empty((t, nh * vd), dtype=self.act_dtype, device=h.device)
-        kernels.heads_gemm(lat.view(t, nh, r), self.uv, o.view(t, nh, vd), nh, scale=gate)
+        kernels.heads_gemm(lat.view(t, nh, r), self.uv, o.view(t, nh, vd), nh, scale=gate, gate=channel)
         return self.o.add_into(o, residual, then_norm)
 
-    def _expanded(self, ctx, q_nope, qa, gate, dense, residual):
+    def _expanded(self, ctx, q_nope, qa, gate, channel, dense, residual):
         """Attention of a prompt step over keys and values expanded per head.  Every head gets rows
         [v | k_nope | k_rot] of its own for the step's tokens (two grouped products from the step's
         latents, the rotated key part copied to every head) and queries [0 | q_nope | q_rot]; the
@@ -187,7 +204,7 @@ class LatentAttention(Part):
         q[:, :, vd + dim:] = qa.view(t, nh, r + rd)[:, :, r:]
         o = torch.empty((t, nh * vd), dtype=self.act_dtype, device=q_nope.device)
         kernels.latent_attention_mma(q.view(t, nh * kd), o, nh, vd, dim + rd, rows, None, 64, ctx.cu_seqlens, ctx.seq_start,
-                                     ctx.seq_slot, ctx.max_new, None, 1, head_stride=hs, out_scale=gate)
+                                     ctx.seq_slot, ctx.max_new, self.window, 1, head_stride=hs, out_scale=gate, out_gate=channel)
         self.o.add_into(o, residual)
 
 

@@ -4,6 +4,7 @@ their projections from.  Not a part itself.
 y[t, o] = sum_i W[o, i] x[t, i] (+ b[o])  (src/kernels.rs:54-57).  The product is written in the
 activation precision, in float32 (logits), or added into the float32 residual stream.  A factor per
 output feature on what is added (``out_scale``, float32 [out]) is applied in float32 after the product.
+``stores``: ``add_into`` writes its rows instead of adding to them (rows that are the product's alone).
 """
 from __future__ import annotations
 
@@ -20,6 +21,7 @@ class Linear:
         self.bias = None if bias is None else bias.to(torch.float32).contiguous()
         self.out_features, self.in_features = weight.shape
         self.out_scale: Optional[torch.Tensor] = None
+        self.stores = False
 
     @classmethod
     def stacked(cls, matrices, bias: Optional[torch.Tensor] = None, multiple: int = 1) -> "Linear":
@@ -48,6 +50,11 @@ class Linear:
         """residual += (x @ W.T (+ b)) * out_scale; residual is float32.  ``then_norm``: the RMSNorm part that
         reads the residual next, if any; where the kernel can it leaves that norm's input
         (kernels.UnscaledRows), which is returned, else None and the norm runs by itself."""
+        if self.stores:
+            if self.out_scale is not None or then_norm is not None:
+                raise ValueError("a product that stores its rows takes no factor on them and leaves nothing for a norm")
+            kernels.gemm(x, self.weight, residual, self.bias)
+            return None
         link = (then_norm.weight, then_norm.eps) if then_norm is not None else None
         return kernels.gemm(x, self.weight, residual, self.bias, accumulate=True, then_norm=link, col_scale=self.out_scale)
 

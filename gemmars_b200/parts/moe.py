@@ -18,8 +18,11 @@ More parameters.  ``gated`` False: an expert has no gate matrix, out = down act(
 and ``e<j>.down``; no clamps, no shared expert.  ``routing`` "softmax_all": the weights are the chosen
 experts' shares of the softmax over all experts, as they are (they do not add up to one); "sigmoid":
 the scores are s = sigmoid(z), the ``top`` largest s + router_bias are chosen, and a chosen expert's
-weight is its s (without the bias) over the sum of the chosen s (+ 1e-20); the default "softmax_top"
-is the softmax over the chosen alone.  ``routing_scale`` (1) multiplies the weights.
+weight is its s (without the bias) over the sum of the chosen s (+ 1e-20); "sigmoid_raw": the same choice,
+the weight s as it is; the default "softmax_top" is the softmax over the chosen alone.  ``routing_scale`` (1)
+multiplies the weights.  ``weigh`` "input": a weight multiplies its expert's input instead of its output,
+the sum of expert(weight * h) (gated experts; applied in float32 to the gate's and up's sums, before the
+activation); the default is "output".
 """
 from __future__ import annotations
 
@@ -53,6 +56,13 @@ class RoutedExperts(Part):
         if not self.gated and (self.activation is None or self.activation not in kernels.PLAIN_ACTS):
             raise ValueError(f"moe: activation {self.activation!r} has no kernel for experts without a gate")
         self.out_scale = None
+        self.stores = False
+        weigh = p.get("weigh", "output")
+        if weigh not in ("output", "input"):
+            raise ValueError(f"moe: weigh must be output or input, got {weigh!r}")
+        self.weigh_input = weigh == "input"
+        if self.weigh_input and not self.gated:
+            raise ValueError("moe: experts without a gate take their weights on the output only")
         if not self.gated and (p.get("shared") or p.get("limit") is not None):
             raise ValueError("moe: experts without a gate take no clamp and no shared expert")
         shared = p.get("shared")
@@ -110,6 +120,10 @@ class RoutedExperts(Part):
         """``scale`` (float32 [hidden]) multiplies what the feed-forward adds."""
         self.out_scale = scale
 
+    def set_output_store(self):
+        """What the feed-forward would add is stored instead."""
+        self.stores = True
+
     def weight_bytes(self):
         """What a decode step of one token reads: the router, ``top`` experts, the shared expert."""
         per = self.gate_up.element_size()
@@ -135,7 +149,8 @@ class RoutedExperts(Part):
                 run = kernels.moe_experts_plain_grouped
             else:
                 run = kernels.moe_experts_plain
-            run(h, idx, wts, self.gate_up, self.down, residual, act=self.activation, col_scale=self.out_scale)
+            run(h, idx, wts, self.gate_up, self.down, residual, act=self.activation, col_scale=self.out_scale,
+                store=self.stores)
             return
         if self.shared_ff and sg is None:
             sg = torch.ones((h.shape[0],), dtype=torch.float32, device=h.device)
@@ -146,7 +161,8 @@ class RoutedExperts(Part):
         else:
             run = kernels.moe_experts
         run(h, idx, wts, sg, self.gate_up, self.down, self.shared_gate_up, self.shared_down, residual,
-            self.limit, self.shared_limit, self.alpha, self.shift, col_scale=self.out_scale)
+            self.limit, self.shared_limit, self.alpha, self.shift, col_scale=self.out_scale,
+            weigh_input=self.weigh_input, store=self.stores)
 
 
 register_part("ffn", "moe", RoutedExperts)

@@ -18,11 +18,11 @@ index whose wavelength makes t turns over ``original`` positions, lo = max(floor
 hi = min(ceil(d(slow)), rotary_dim - 1), the frequency is f / factor * r + f (1 - r) with
 r = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), and the cosines and sines are multiplied by
 ``magnitude`` = 0.1 ln(factor) + 1 (1 without this form).  Only kernels that take a magnitude can
-use such a part (``capped_attention`` does; the fused kernels of ``attention`` do not).
+use such a part (``capped_attention`` and ``latent_attention`` do; the fused kernels of ``attention`` do not).
 
 The attention part fuses the "half" rotation into its q/k kernel when its position encoding is
-this class, and the latent attention part the "interleaved" one into the kernel that writes its
-cache rows; ``apply`` is the stand-alone form of either."""
+this class, the capped and the latent attention parts either layout into the kernels that write
+their cache; ``apply`` is the stand-alone form (of the half layout without a magnitude)."""
 from __future__ import annotations
 
 import math
@@ -115,13 +115,13 @@ class Rotary(Part):
 
     def apply(self, ctx, q, k):
         """Rotates q [T, nh, hd] and k [T, nkv, hd] (contiguous views) in place."""
-        if self.magnitude != 1.0:
-            raise ValueError("rotary: the stand-alone rotation takes no magnitude (use a mixer whose kernel does)")
+        if self.magnitude != 1.0 and self.layout == "half":
+            raise ValueError("rotary: the stand-alone rotation of halves takes no magnitude (use a mixer whose kernel does)")
         for x in (q, k):
             t, heads, hd = x.shape
             if self.layout == "interleaved":
                 if self.rotary_dim:
-                    kernels.rope_pairs(x, ctx.tok_pos, self.inv_freq(x.device), self.rotary_dim)
+                    kernels.rope_pairs(x, ctx.tok_pos, self.inv_freq(x.device), self.rotary_dim, self.magnitude)
                 continue
             flat = x.view(t, heads * hd)
             # all heads are treated as "q" heads of one tensor: rotate in place, scale 1
