@@ -1,2 +1,2 @@
 """Architectures.  Importing this package registers each of them under its config.json names."""
-from . import dalerax, kuporax, mevuvik, nogosun, qwen3, toretar  # noqa: F401
+from . import dalerax, fezozen, kuporax, mevuvik, nogosun, qwen3, toretar  # noqa: F401
