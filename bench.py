@@ -2,7 +2,7 @@
 """Decode and prefill throughput of Qwen3-shaped models with random weights on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl reference] [--config 8b|4b|32b]
-    python bench.py --compare toretar|kuporax|dalerax|nogosun|mevuvik [--sizes small,lite,mid] [--batch 8] [--context 4096]
+    python bench.py --compare toretar|kuporax|dalerax|nogosun|mevuvik|fezozen [--sizes small,lite,mid] [--batch 8] [--context 4096]
 
 ``--config 8b`` (the default) is the headline benchmark.  A step is one decode step of a batch
 of 8 sequences at a context of 8,192 tokens.  One JSON line is printed: ``value`` = decoded
@@ -329,6 +329,35 @@ def mevuvik_prefill_flops(cfg, t):
     return total + 2 * w * cfg["vocab"]
 
 
+def fezozen_prefill_flops(cfg, t):
+    """Floating-point operations of a prompt of ``t`` tokens from position 0 (a layer that runs another
+    layer's tensors counts like one of its own): every product, the latent attention as the engine takes
+    it (toretar_prefill_flops), scores and weighted values over the keys each token's mask lets it see,
+    the router and the chosen experts (three matrices)."""
+    import torch
+    from gemmars_b200 import kernels
+    w, total = cfg["width"], 0
+    for layer in cfg["layers"]:
+        m, mlp = layer["mixer"], layer.get("mlp")
+        nh, dim, vd = m["heads"], m["dim"], m["vdim"]
+        size = (m.get("mask") or {}).get("size", t)
+        seen = sum(min(p + 1, size) for p in range(t))
+        if layer["type"] == "latent_attention":
+            rd, r = m["rot_dim"], m["kv_rank"]
+            per_token = 2 * (w * (nh * (dim + rd) + r + rd + nh * vd) + nh * vd * w) + 2 * nh * (dim + vd) * r
+            if t >= kernels.LATENT_EXPAND_MIN_TOKENS and kernels.latent_expand_usable(torch.bfloat16, r, dim, rd, vd):
+                attention = 2 * nh * (dim + rd + vd) * seen
+            else:
+                attention = 2 * nh * (2 * r + rd) * seen
+        else:
+            per_token = 2 * w * (nh * dim + m["kv_heads"] * (dim + vd)) + 2 * nh * vd * w
+            attention = 2 * nh * (dim + vd) * seen
+        if mlp is not None:
+            per_token += 2 * w * mlp["router"]["experts"] + 6 * w * mlp["router"]["top"] * mlp["expert"]["ff"]
+        total += per_token * t + attention
+    return total + 2 * w * cfg["vocab"]
+
+
 def fill_cache(runner, slots, length, real, vocab, gen):
     """Brings every slot to ``length`` cached tokens: by running prompts (real) or by
     reserving the pages and writing random keys and values (synthetic)."""
@@ -426,6 +455,8 @@ def time_prefill(eng, cfg, tokens, tflops, tflops_sustained):
         flops = nogosun_prefill_flops(cfg, tokens)
     elif cfg.get("architecture") == "Mevuvik":
         flops = mevuvik_prefill_flops(cfg, tokens)
+    elif cfg.get("architecture") == "Fezozen":
+        flops = fezozen_prefill_flops(cfg, tokens)
     elif cfg.get("sliding_window") and cfg.get("use_sliding_window"):
         size = cfg["sliding_window"]      # a window on every layer: the keys a token sees, not the causal half
         seen = sum(min(p + 1, size) for p in range(tokens))
@@ -618,11 +649,11 @@ def kernel_table(eng, tokens, batch, context):
 def run_compare(args):
     """Prompt and decode throughput of models of one architecture beside models of another with the
     same width, depth and per-token feed-forward size (Toretar and Kuporax beside Qwen3, Dalerax
-    beside Kuporax, Nogosun beside Dalerax, Mevuvik beside Nogosun), with a table of each one's kernels."""
-    from gemmars_b200.tuning import DALERAX_PAIRS, KUPORAX_PAIRS, MEVUVIK_PAIRS, NOGOSUN_PAIRS, PAIRS
+    beside Kuporax, Nogosun beside Dalerax, Mevuvik beside Nogosun, Fezozen beside Toretar), with a table of each one's kernels."""
+    from gemmars_b200.tuning import DALERAX_PAIRS, FEZOZEN_PAIRS, KUPORAX_PAIRS, MEVUVIK_PAIRS, NOGOSUN_PAIRS, PAIRS
     pairs = {"kuporax": KUPORAX_PAIRS, "dalerax": DALERAX_PAIRS, "nogosun": NOGOSUN_PAIRS,
-             "mevuvik": MEVUVIK_PAIRS}.get(args.compare, PAIRS)
-    beside = {"dalerax": "kuporax", "nogosun": "dalerax", "mevuvik": "nogosun"}.get(args.compare, "qwen3")
+             "mevuvik": MEVUVIK_PAIRS, "fezozen": FEZOZEN_PAIRS}.get(args.compare, PAIRS)
+    beside = {"dalerax": "kuporax", "nogosun": "dalerax", "mevuvik": "nogosun", "fezozen": "toretar"}.get(args.compare, "qwen3")
     hbm_gbs, tflops, tflops_sustained, peak_src = peaks()
     sizes = [s for s in args.sizes.split(",") if s]
     out = {}
@@ -661,9 +692,9 @@ def main():
     ap.add_argument("--e2e-tokens", type=int, default=E2E_TOKENS,
                     help="tokens a sequence generates in the end-to-end run (fewer for runs under a profiler)")
     ap.add_argument("--options", default="", help='further engine options, "key=value;key=value"')
-    ap.add_argument("--compare", choices=["toretar", "kuporax", "dalerax", "nogosun", "mevuvik"], default=None,
+    ap.add_argument("--compare", choices=["toretar", "kuporax", "dalerax", "nogosun", "mevuvik", "fezozen"], default=None,
                     help="instead of the headline: models of that architecture beside ones of equal size (Qwen3-shaped; "
-                         "Kuporax-shaped for dalerax; Dalerax-shaped for nogosun; Nogosun-shaped for mevuvik)")
+                         "Kuporax-shaped for dalerax; Dalerax-shaped for nogosun; Nogosun-shaped for mevuvik; Toretar-shaped for fezozen)")
     ap.add_argument("--sizes", default="small,lite,mid", help="with --compare: which pairs of tuning.PAIRS")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -225,6 +225,52 @@ for _name, (_m, _n) in MEVUVIK_PAIRS.items():
     PAIR_SHAPES[f"mevuvik-{_name}"] = (f"Mevuvik shape '{_name}'", _m)
 
 
+def fezozen_shape(width, ff, heads, window, rank, experts, top, order=("attention_2", "attention", "latent_attention", "attention_2"),
+                  vocab=102400):
+    """A Fezozen config.json object: attention over every key (``heads`` heads of 128, a quarter as many
+    kv heads, half of every head turned with scaling, capped scores), windowed attention with unit q and
+    k (the same heads, every dim turned), the second of which runs the first one's tensors again, and
+    windowed latent attention (``heads`` heads of 128 + 64 with values of 128).  Every layer routes
+    ``top`` of ``experts`` gated experts, sized so that a token passes ``ff`` hidden units in all."""
+    heads_128 = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    stretched = {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+    mixers = {
+        "attention": {**heads_128, "softcap": 30.0, "rot": {"base": 1000000.0, "dims": 64, "scaling": stretched}},
+        "attention_2": {**heads_128, "mask": {"size": window}, "rot": {"base": 1000000.0, "dims": 128}},
+        "latent_attention": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": rank, "scale": 192 ** -0.5,
+                             "mask": {"size": window}, "rot": {"base": 1000000.0, "dims": 64, "scaling": stretched}},
+    }
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff // top}}
+    layers, first = [], {}
+    for i, kind in enumerate(order):
+        layer = {"type": kind, "mixer": mixers[kind], "mlp": mlp}
+        if kind in first:
+            layer["weights_of"] = first[kind]
+        first.setdefault(kind, i)
+        layers.append(layer)
+    return {"architecture": "Fezozen", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "layers": layers}
+
+
+# Fezozen beside Toretar, the nearest design the package has (softmax attention alone, pairs turned side by
+# side, latent attention with a gate, gated experts): the same width, layers, vocabulary, heads, latent and
+# hidden units a token passes (Toretar's through one expert fewer and a shared expert as wide as one).  Its
+# grouped-query attention's like is the capped attention of Nogosun ("nogosun-*").
+def _fezozen_pair(width, ff, heads, window, rank, experts, top):
+    return (fezozen_shape(width, ff, heads, window, rank, experts, top),
+            toretar_shape(4, width, heads, 128, 64, 128, rank, experts, top - 1, ff // top, ff // top))
+
+
+FEZOZEN_PAIRS = {
+    "small": _fezozen_pair(1024, 4096, 8, 512, 256, 16, 4),
+    "lite": _fezozen_pair(2048, 8192, 16, 1024, 512, 32, 4),
+    "mid": _fezozen_pair(4096, 12288, 32, 2048, 512, 32, 4),
+}
+for _name, (_f, _t) in FEZOZEN_PAIRS.items():
+    PAIR_SHAPES[f"fezozen-{_name}"] = (f"Fezozen shape '{_name}'", _f)
+    PAIR_SHAPES[f"beside-fezozen-{_name}"] = (f"Toretar shape beside Fezozen '{_name}'", _t)
+
+
 def random_engine(cfg, max_batch, cache_tokens, options=""):
     """An engine over random weights of ``cfg`` made on the device; the tensors are taken out of
     their dict as they are bound, so that a model of 65 GB and its stacked q/k/v and gate/up copies

@@ -388,3 +388,82 @@ MEVUVIK_C = {
         {"type": "parallel", "mixer": _mevuvik_pair((2, 1, 20, 12, 0.22), (3, 7, 9, 4.0), 1.0, 1.0), "mlp": None},
     ],
 }
+
+
+# ---------------------------------------------------------------------------------------------- Fezozen
+def _fezozen_rot(base, dims, scaling=None):
+    rot = {"base": base, "dims": dims}
+    if scaling is not None:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return rot
+
+
+def _fezozen_attention(heads, kv_heads, dim, vdim, scale, cap, rot):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "rot": rot}
+    if cap is not None:
+        m["softcap"] = cap
+    return m
+
+
+def _fezozen_unit(heads, kv_heads, dim, vdim, scale, size, rot):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": size}, "rot": rot}
+
+
+def _fezozen_latent(heads, dim, rot_dim, vdim, kv_rank, scale, size, base, scaling=None):
+    return {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "scale": scale,
+            "mask": {"size": size}, "rot": _fezozen_rot(base, rot_dim, scaling)}
+
+
+def _fezozen_moe(experts, top, ff):
+    return {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff}}
+
+
+_FA_UNIT = _fezozen_unit(6, 2, 20, 12, 0.5, 20, _fezozen_rot(300.0, 12))
+_FA_LATENT = _fezozen_latent(3, 24, 12, 20, 44, 0.2, 33, 500.0, (4.0, 64, 8.0, 0.5))
+
+# Small sizes that no tensor-core attention takes but the products do (a width of 72): windows of 20 and
+# 33, half-rotated heads, keys wider and narrower than values, a latent layer without feed-forward that
+# runs twice and a windowed layer that runs twice, every expert chosen in one layer.
+FEZOZEN_A = {
+    "architecture": "Fezozen", "vocab": 211, "width": 72, "embedding": {"scale": 3.0}, "norm": {"eps": 1e-5},
+    "layers": [
+        {"type": "attention_2", "mixer": _FA_UNIT, "mlp": _fezozen_moe(5, 2, 40)},
+        {"type": "latent_attention", "mixer": _FA_LATENT, "mlp": None},
+        {"type": "attention", "mixer": _fezozen_attention(4, 4, 24, 28, 0.2, 3.0, _fezozen_rot(500.0, 16, (4.0, 64, 8.0, 0.5))),
+         "mlp": _fezozen_moe(4, 4, 32)},
+        {"type": "latent_attention", "mixer": _FA_LATENT, "mlp": None, "weights_of": 1},
+        {"type": "attention_2", "mixer": _FA_UNIT, "mlp": _fezozen_moe(5, 2, 40), "weights_of": 0},
+        {"type": "attention", "mixer": _fezozen_attention(3, 1, 20, 24, 0.25, 4.0, _fezozen_rot(1e4, 20, (2.5, 100, 4.0, 1.0))),
+         "mlp": _fezozen_moe(3, 1, 48)},
+    ],
+}
+
+_FB_CAPPED = _fezozen_attention(8, 2, 64, 40, 0.125, 25.0, _fezozen_rot(1e5, 32, (8.0, 128, 16.0, 1.0)))
+
+# Sizes the tensor cores take: capped attention with keys of 64 and values of 40, unit q and k under a
+# window one longer than a page, latents of 112 + 16 under a window of 100 (expanded per head in long
+# prompts) and of 64 + 32 under a window of exactly a page (not expanded).
+FEZOZEN_B = {
+    "architecture": "Fezozen", "vocab": 520, "width": 128, "embedding": {"scale": 9.0}, "norm": {"eps": 1e-6},
+    "layers": [
+        {"type": "latent_attention", "mixer": _fezozen_latent(6, 16, 16, 32, 112, 0.18, 100, 1e5, (4.0, 128, 8.0, 1.0)),
+         "mlp": _fezozen_moe(8, 3, 64)},
+        {"type": "attention", "mixer": _FB_CAPPED, "mlp": _fezozen_moe(6, 1, 96)},
+        {"type": "attention_2", "mixer": _fezozen_unit(6, 2, 32, 64, 0.25, 65, _fezozen_rot(1e4, 32)), "mlp": _fezozen_moe(8, 3, 64)},
+        {"type": "latent_attention", "mixer": _fezozen_latent(4, 32, 32, 64, 64, 0.125, 64, 1e4), "mlp": _fezozen_moe(6, 2, 72)},
+        {"type": "attention", "mixer": _FB_CAPPED, "mlp": _fezozen_moe(6, 1, 96), "weights_of": 1},
+    ],
+}
+
+# A width that is no multiple of 8 and heads that are no multiple of 16 (plain kernels throughout in
+# bfloat16): a window of a single key, one kv head and one latent head, no cap, no rotation in one layer
+# and two rotated dims in another, an embedding that is not scaled, a single expert.
+FEZOZEN_C = {
+    "architecture": "Fezozen", "vocab": 97, "width": 52, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+    "layers": [
+        {"type": "attention", "mixer": _fezozen_attention(2, 2, 20, 20, 0.22, None, _fezozen_rot(50.0, 0)), "mlp": _fezozen_moe(1, 1, 20)},
+        {"type": "latent_attention", "mixer": _fezozen_latent(1, 6, 10, 5, 11, 0.25, 9, 50.0), "mlp": _fezozen_moe(4, 2, 12)},
+        {"type": "attention_2", "mixer": _fezozen_unit(3, 1, 12, 20, 0.6, 17, _fezozen_rot(50.0, 2)), "mlp": None},
+        {"type": "attention_2", "mixer": _fezozen_unit(2, 1, 12, 9, 0.6, 1, _fezozen_rot(50.0, 12)), "mlp": _fezozen_moe(3, 3, 28)},
+    ],
+}
