@@ -1,8 +1,15 @@
 // bfloat16 causal grouped-query attention of packed prompts on the 5th-generation tensor cores
-// (tcgen05, sm_100a), for head sizes 64 and 128.  Compiled for one head size (-DGB_HEAD_DIM=...).
+// (tcgen05, sm_100a).  Compiled for one size of keys (-DGB_HEAD_DIM=..., a multiple of 8 up to 128) and
+// one of values (-DGB_VALUE_DIM=..., a multiple of 16 up to 128; the keys' size by default).
 //
 // Mathematics as everywhere (src/model.rs:1187-1226, src/kernels.rs:1550-1561): the query at
-// position p sees the keys lo..p of its own sequence, softmax in float32, o = sum p_j V[j].
+// position p sees the keys lo..p of its own sequence, softmax in float32, o = sum p_j V[j].  The scores
+// may be scaled and capped (cap tanh(score / cap), the hardware's tanh as in attention_capped_mma.cu), a
+// sink per head may join the softmax's denominator, and a sigmoid gate per number or per head may
+// multiply the result.
+//
+// Keys that are no multiple of 64 wide are padded in shared memory: TMA fills the key tile's columns past
+// the row with zeros, and whatever the query tile holds there (the next head's dims) counts nothing.
 //
 // A CTA owns 128 consecutive tokens of one sequence for one query head and walks the cache one
 // page (64 keys) at a time:
@@ -21,17 +28,22 @@
 #ifndef GB_HEAD_DIM
 #define GB_HEAD_DIM 128
 #endif
+#ifndef GB_VALUE_DIM
+#define GB_VALUE_DIM GB_HEAD_DIM
+#endif
 
 namespace {
 
-constexpr int HD = GB_HEAD_DIM;
-static_assert(HD == 64 || HD == 128, "the tensor-core prefill kernel takes head sizes 64 and 128");
-constexpr int ROWS = 128, KEYS = 64, QH = HD / 64;
-constexpr uint32_t Q_BYTES = ROWS * HD * 2, K_BYTES = KEYS * HD * 2, V_BYTES = HD * KEYS * 2, P_BYTES = ROWS * KEYS * 2;
+constexpr int HD = GB_HEAD_DIM, VD = GB_VALUE_DIM;
+static_assert(HD % 8 == 0 && HD >= 8 && HD <= 128, "keys: a multiple of 8 up to 128 (a head starts on a 16-byte boundary)");
+static_assert(VD % 16 == 0 && VD >= 16 && VD <= 128, "values: a multiple of 16 up to 128");
+constexpr int ROWS = 128, KEYS = 64, QH = (HD + 63) / 64, HDP = QH * 64;     // HDP: a key's row in shared memory
+constexpr uint32_t Q_BYTES = ROWS * HDP * 2, K_BYTES = KEYS * HDP * 2, V_BYTES = VD * KEYS * 2, P_BYTES = ROWS * KEYS * 2;
+constexpr int OC = VD % 32 == 0 ? 32 : 16;                                    // columns of O a thread handles at a time
 constexpr uint32_t SMEM_TILES = Q_BYTES + 2 * K_BYTES + 2 * V_BYTES + P_BYTES;
 constexpr uint32_t TMEM_COLS = 256, S_COL0 = 0, S_COL1 = 64, O_COL = 128;
 constexpr uint32_t IDESC_S = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(KEYS >> 3) << 17) | ((uint32_t)(ROWS >> 4) << 24);
-constexpr uint32_t IDESC_PV = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(HD >> 3) << 17) | ((uint32_t)(ROWS >> 4) << 24);
+constexpr uint32_t IDESC_PV = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(VD >> 3) << 17) | ((uint32_t)(ROWS >> 4) << 24);
 constexpr float RESCALE_STEP = 8.0f;   // how far a row's maximum may outgrow its reference before O is rescaled
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -56,6 +68,19 @@ __device__ __forceinline__ void tc_st32(uint32_t taddr, const uint32_t* v) {
         "r"(v[18]), "r"(v[19]), "r"(v[20]), "r"(v[21]), "r"(v[22]), "r"(v[23]), "r"(v[24]), "r"(v[25]), "r"(v[26]),
         "r"(v[27]), "r"(v[28]), "r"(v[29]), "r"(v[30]), "r"(v[31])
       : "memory");
+}
+__device__ __forceinline__ void tc_st16(uint32_t taddr, const uint32_t* v) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
+      ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]),
+        "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15])
+      : "memory");
+}
+template <int N> __device__ __forceinline__ void tc_ld_cols(uint32_t taddr, uint32_t* v) {
+  if constexpr (N == 32) tc_ld32(taddr, v); else tc_ld16(taddr, v);
+}
+template <int N> __device__ __forceinline__ void tc_st_cols(uint32_t taddr, const uint32_t* v) {
+  if constexpr (N == 32) tc_st32(taddr, v); else tc_st16(taddr, v);
 }
 __device__ __forceinline__ void tc_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
@@ -86,13 +111,30 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
   return *(uint32_t*)&v;
 }
 
+__device__ __forceinline__ float tanh_fast(float x) {
+  float y;
+  asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// What happens to the scores and to the result beside the softmax.  A score in log2 units is
+// mul * (q . k), or with a cap mul * tanh(pre * (q . k)); mul is positive.
+struct Extras {
+  float mul = LOG2E, pre = 0.f;
+  const float* sink = nullptr;                                        // per head, natural units
+  const bf16* gate = nullptr; long long gate_stride = 0; int gate_per_head = 0;
+  float out_scale = 1.f;
+};
+
 // grid (query heads, token tiles upper bound); block 192: warps 0-3 softmax, 4 TMA, 5 MMA.
+template <bool CAP>
 __global__ void __launch_bounds__(192, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, long long out_stride,
                             const int* __restrict__ page_table, int table_width, int nkv,
                             const int* __restrict__ cu_seqlens, const int* __restrict__ seq_start,
-                            const int* __restrict__ seq_slot, int n_seqs, int nh, int window) {
+                            const int* __restrict__ seq_slot, int n_seqs, int nh, int window,
+                            const __grid_constant__ Extras ex) {
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t* q_smem = smem;
   uint8_t* k_smem = q_smem + Q_BYTES;          // two stages
@@ -196,7 +238,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           const int page = page_table[(size_t)slot * table_width + (kt_begin + jv) % table_width];
           const int row = page * nkv + kvh;
           mbar_expect_tx(&v_full[sidx], V_BYTES);
-          tma_load_2d(v_smem + sidx * V_BYTES, &map_v, 0, row * HD, &v_full[sidx]);
+          tma_load_2d(v_smem + sidx * V_BYTES, &map_v, 0, row * VD, &v_full[sidx]);
           ++jv;
           moved = true;
         }
@@ -279,6 +321,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[sb]);     // this warp has its rows of S: the buffer may be written again
       const int key0 = (kt_begin + j) * KEYS;
+      if (CAP) {
+#pragma unroll
+        for (int c = 0; c < 64; ++c) sv[c] = __float_as_uint(tanh_fast(__uint_as_float(sv[c]) * ex.pre));
+      }
       // Only the pages on the diagonal and at a window's lower edge hold keys that a row must not
       // see; the others skip the two comparisons and the select per score (the loop is bound by
       // the number of instructions the four softmax warps issue, not by the exponentials).
@@ -297,7 +343,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         mx2 = fmaxf(mx2, __uint_as_float(sv[c + 2]));
         mx3 = fmaxf(mx3, __uint_as_float(sv[c + 3]));
       }
-      const float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * LOG2E;   // log2 units from here on
+      const float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * ex.mul;   // log2 units from here on
       // m is the reference the exponentials are taken against, not always the running maximum: it
       // moves only when the maximum has outgrown it by more than RESCALE_STEP (in log2 units), so
       // that O, which would have to be rescaled with it, is left alone on most pages.  p can then
@@ -311,10 +357,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       uint32_t pk[32];
 #pragma unroll
       for (int c = 0; c < 32; ++c) {
-        // one multiply-add and one ex2 per score: 2^(s * log2(e) - reference); a masked score is
+        // one multiply-add and one ex2 per score: 2^(s * mul - reference); a masked score is
         // -inf and gives 0
-        const float a = ex2(fmaf(__uint_as_float(sv[2 * c]), LOG2E, -u));
-        const float bq = ex2(fmaf(__uint_as_float(sv[2 * c + 1]), LOG2E, -u));
+        const float a = ex2(fmaf(__uint_as_float(sv[2 * c]), ex.mul, -u));
+        const float bq = ex2(fmaf(__uint_as_float(sv[2 * c + 1]), ex.mul, -u));
         sum0 += a;
         sum1 += bq;
         pk[c] = pack2(a, bq);
@@ -327,13 +373,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         tc_fence_after();
         if (__any_sync(0xffffffffu, alpha != 1.0f)) {
 #pragma unroll 1
-          for (int c = 0; c < HD; c += 32) {
-            uint32_t ov[32];
-            tc_ld32(lane_addr + O_COL + c, ov);
+          for (int c = 0; c < VD; c += OC) {
+            uint32_t ov[OC];
+            tc_ld_cols<OC>(lane_addr + O_COL + c, ov);
             tc_wait_ld();
 #pragma unroll
-            for (int i = 0; i < 32; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * alpha);
-            tc_st32(lane_addr + O_COL + c, ov);
+            for (int i = 0; i < OC; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * alpha);
+            tc_st_cols<OC>(lane_addr + O_COL + c, ov);
           }
           tc_wait_st();
         }
@@ -351,16 +397,29 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (ok) ok = __all_sync(0xffffffffu, wait_or_abort(o_done, (n_tiles - 1) & 1, abort, 6));
     if (ok) {
       tc_fence_after();
-      const float inv = l > 0.f ? 1.0f / l : 0.f;
-      bf16* dst = out + (size_t)(tok0 + r) * out_stride + (size_t)head * HD;
+      float keep = ex.out_scale;
+      if (ex.sink && m > -INFINITY) {       // exp(sink) joins the denominator: both sides against the larger reference
+        const float s2 = ex.sink[head] * LOG2E, top = fmaxf(m, s2), share = exp2f(m - top);
+        l = l * share + exp2f(s2 - top);
+        keep *= share;
+      }
+      float inv = l > 0.f ? keep / l : 0.f;
+      const bf16* gt = ex.gate && valid ? ex.gate + (size_t)(tok0 + r) * ex.gate_stride : nullptr;
+      if (gt && ex.gate_per_head) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(gt[head])));
+      bf16* dst = out + (size_t)(tok0 + r) * out_stride + (size_t)head * VD;
 #pragma unroll 1
-      for (int c = 0; c < HD; c += 32) {
-        uint32_t ov[32];
-        tc_ld32(lane_addr + O_COL + c, ov);
+      for (int c = 0; c < VD; c += OC) {
+        uint32_t ov[OC];
+        tc_ld_cols<OC>(lane_addr + O_COL + c, ov);
         tc_wait_ld();
         if (valid) {
+          if (gt && !ex.gate_per_head) {
 #pragma unroll
-          for (int i = 0; i < 4; ++i) {
+            for (int i = 0; i < OC; ++i)
+              ov[i] = __float_as_uint(__uint_as_float(ov[i]) / (1.0f + __expf(-__bfloat162float(gt[head * VD + c + i]))));
+          }
+#pragma unroll
+          for (int i = 0; i < OC / 8; ++i) {
             uint4 w;
             w.x = pack2(__uint_as_float(ov[8 * i]) * inv, __uint_as_float(ov[8 * i + 1]) * inv);
             w.y = pack2(__uint_as_float(ov[8 * i + 2]) * inv, __uint_as_float(ov[8 * i + 3]) * inv);
@@ -380,35 +439,61 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 
 }  // namespace
 
-// q, out: [ntok, nh * HD] bfloat16, tokens of all sequences packed (cu_seqlens: [n_seqs + 1]); q rows
-// q_stride elements apart.  kcache: [pages, nkv, 64, HD]; vcache: [pages, nkv, HD, 64] (pages counts
-// every page of the layer, the spare one included).  seq_start: cache length of each sequence before
-// this step; the cache already holds this step's keys and values.
-GB_EXPORT int gb_attention_prefill_tc(const void* q, long long q_stride, void* out, long long out_stride,
-                                      const void* kcache, const void* vcache, long long pages, const int* page_table,
-                                      int table_width, int page_size, int nkv, int hd, const int* cu_seqlens,
-                                      const int* seq_start, const int* seq_slot, int n_seqs, int ntok, int nh,
-                                      int window, cudaStream_t stream) {
+// q: [ntok, nh * HD], out: [ntok, nh * VD] bfloat16, tokens of all sequences packed (cu_seqlens: [n_seqs +
+// 1]); q rows q_stride elements apart.  kcache: [pages, nkv, 64, HD]; vcache: [pages, nkv, VD, 64] (pages
+// counts every page of the layer, the spare one included).  seq_start: cache length of each sequence
+// before this step; the cache already holds this step's keys and values.  score = (q . k) * scale (positive),
+// capped when cap > 0; sink: float32 [nh] or null; gate: bfloat16 [ntok, nh * VD], with gate_per_head [ntok,
+// nh], rows gate_stride elements apart, or null; the result times out_scale.
+GB_EXPORT int gb_attention_prefill_tc_ext(const void* q, long long q_stride, void* out, long long out_stride,
+                                          const void* kcache, const void* vcache, long long pages, const int* page_table,
+                                          int table_width, int page_size, int nkv, int hd, int vd, const int* cu_seqlens,
+                                          const int* seq_start, const int* seq_slot, int n_seqs, int ntok, int nh,
+                                          int window, float scale, float cap, const float* sink, const void* gate,
+                                          long long gate_stride, int gate_per_head, float out_scale, cudaStream_t stream) {
   if (ntok <= 0 || n_seqs <= 0) return 0;
-  if (hd != HD || page_size != KEYS || nkv <= 0 || nh % nkv || pages <= 0) return GB_ERR_SIZE;
+  if (!(scale > 0.f)) return GB_ERR_ARG;
+  if (hd != HD || vd != VD || page_size != KEYS || nkv <= 0 || nh % nkv || pages <= 0) return GB_ERR_SIZE;
   if (((uintptr_t)q & 15) || (q_stride % 8) || ((uintptr_t)out & 15) || (out_stride % 8) || ((uintptr_t)kcache & 15) ||
       ((uintptr_t)vcache & 15))
     return GB_ERR_SIZE;
   CUtensorMap mq, mk, mv;
   if (!tensor_map(&mq, q, (uint64_t)ntok, (uint64_t)nh * HD, (uint64_t)q_stride * 2, ROWS)) return GB_ERR_ARG;
   if (!tensor_map(&mk, kcache, (uint64_t)pages * nkv * KEYS, (uint64_t)HD, (uint64_t)HD * 2, KEYS)) return GB_ERR_ARG;
-  if (!tensor_map(&mv, vcache, (uint64_t)pages * nkv * HD, (uint64_t)KEYS, (uint64_t)KEYS * 2, HD)) return GB_ERR_ARG;
+  if (!tensor_map(&mv, vcache, (uint64_t)pages * nkv * VD, (uint64_t)KEYS, (uint64_t)KEYS * 2, VD)) return GB_ERR_ARG;
   constexpr size_t SMEM = SMEM_TILES + 15 * 8 + 16;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess)
+    if (cudaFuncSetAttribute(attention_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess)
       return (int)cudaGetLastError();
     configured = true;
   }
+  Extras ex;
+  ex.mul = (cap > 0.f ? cap : scale) * LOG2E;
+  ex.pre = cap > 0.f ? scale / cap : 0.f;
+  ex.sink = sink;
+  ex.gate = (const bf16*)gate; ex.gate_stride = gate_stride; ex.gate_per_head = gate_per_head;
+  ex.out_scale = out_scale;
   dim3 grid(nh, (ntok + ROWS - 1) / ROWS + n_seqs);
-  gb_launch(attention_prefill_tc_kernel, grid, 192, SMEM, stream, mq, mk, mv, (bf16*)out, out_stride, page_table,
-            table_width, nkv, cu_seqlens, seq_start, seq_slot, n_seqs, nh, window);
+  if (cap > 0.f)
+    gb_launch(attention_prefill_tc_kernel<true>, grid, 192, SMEM, stream, mq, mk, mv, (bf16*)out, out_stride, page_table,
+              table_width, nkv, cu_seqlens, seq_start, seq_slot, n_seqs, nh, window, ex);
+  else
+    gb_launch(attention_prefill_tc_kernel<false>, grid, 192, SMEM, stream, mq, mk, mv, (bf16*)out, out_stride, page_table,
+              table_width, nkv, cu_seqlens, seq_start, seq_slot, n_seqs, nh, window, ex);
   return gb_launch_status();
+}
+
+// The same for queries that carry their scale, keys and values of one size, nothing else.
+GB_EXPORT int gb_attention_prefill_tc(const void* q, long long q_stride, void* out, long long out_stride,
+                                      const void* kcache, const void* vcache, long long pages, const int* page_table,
+                                      int table_width, int page_size, int nkv, int hd, const int* cu_seqlens,
+                                      const int* seq_start, const int* seq_slot, int n_seqs, int ntok, int nh,
+                                      int window, cudaStream_t stream) {
+  return gb_attention_prefill_tc_ext(q, q_stride, out, out_stride, kcache, vcache, pages, page_table, table_width, page_size,
+                                     nkv, hd, hd, cu_seqlens, seq_start, seq_slot, n_seqs, ntok, nh, window, 1.0f, 0.f,
+                                     nullptr, nullptr, 0, 0, 1.0f, stream);
 }
 
 // 0, or the code of the first bounded wait that ran out (synchronizes the device).

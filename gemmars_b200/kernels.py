@@ -1941,8 +1941,23 @@ def attention_capped_mma_usable(dtype, dim: int, vdim: int, page_size: int) -> b
             and page_size % 32 == 0)
 
 
+#: prompts that bring at least this many tokens a sequence take the tcgen05 kernel where its sizes allow
+CAPPED_TC_MIN_TOKENS = 32
+
+
+def attention_capped_tc_usable(dtype, dim: int, vdim: int, page_size: int) -> bool:
+    return (dtype == torch.bfloat16 and dim % 8 == 0 and 8 <= dim <= 128 and vdim % 16 == 0 and 16 <= vdim <= 128
+            and page_size == 64)
+
+
+def _prefill_tc_defines(dim: int, vdim: int):
+    return (("GB_HEAD_DIM", dim),) + ((("GB_VALUE_DIM", vdim),) if vdim != dim else ())
+
+
 def attention_capped_units(compute: str, dim: int, vdim: int, page_size: int = 64):
     units = [("attention_capped", ())]
+    if compute == "bfloat16" and attention_capped_tc_usable(torch.bfloat16, dim, vdim, page_size):
+        units.append(("attention_prefill_tc", _prefill_tc_defines(dim, vdim)))
     if compute == "bfloat16" and attention_capped_mma_usable(torch.bfloat16, dim, vdim, page_size):
         units.append(("attention_capped_mma", (("GB_HEAD_DIM", dim), ("GB_VALUE_DIM", vdim))))
     return units
@@ -1956,8 +1971,10 @@ def attention_capped(ctx, q, out, heads, kcache, vcache, page_table, page_size, 
     sequence stay visible; ``sink`` (float32 [heads]): exp(sink[head]) is one more term of the
     softmax's denominator; the output times sigmoid(gate) * out_scale, ``gate`` [T, heads * vdim] or with
     ``gate_per_head`` [T, heads].  bfloat16
-    steps run on the tensor cores where the sizes allow (keys a multiple of 16, values of 8, up to
-    256), prompts and single tokens alike; float32 and other sizes run the plain kernel."""
+    steps run on the tensor cores where the sizes allow: prompts without kept first keys on the tcgen05
+    kernel of plain attention (keys a multiple of 8, values of 16, up to 128), the rest, single tokens
+    included, on mma.sync (keys a multiple of 16, values of 8, up to 256); float32 and other sizes run
+    the plain kernel."""
     _cuda(q, out, kcache, vcache, page_table, gate, sink)
     groups, dim, vdim = kcache.shape[1], kcache.shape[3], vcache.shape[2]
     assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == heads)
@@ -1968,6 +1985,19 @@ def attention_capped(ctx, q, out, heads, kcache, vcache, page_table, page_size, 
     assert q.dtype == out.dtype == kcache.dtype == vcache.dtype and (gate is None or gate.dtype == q.dtype)
     assert q.shape[1] == heads * dim and out.shape[1] == heads * vdim
     assert gate is None or gate.shape[1] >= (heads if gate_per_head else heads * vdim)
+    if (CAPPED_ATTENTION_MMA and attention_capped_tc_usable(q.dtype, dim, vdim, page_size)
+            and getattr(ctx, "max_new", 0) >= CAPPED_TC_MIN_TOKENS and (keep_first == 0 or not window) and scale > 0.0
+            and qp % 16 == 0 and ldq % 8 == 0 and op % 16 == 0 and ldo % 8 == 0):
+        f = _fn("attention_prefill_tc", "gb_attention_prefill_tc_ext",
+                [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int,
+                 c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p,
+                 c_longlong, c_int, c_float, c_void_p], defines=_prefill_tc_defines(dim, vdim))
+        _check(f(qp, ldq, op, ldo, kcache.data_ptr(), vcache.data_ptr(), kcache.shape[0], page_table.data_ptr(),
+                 page_table.shape[1], page_size, groups, dim, vdim, ctx.cu_seqlens.data_ptr(), ctx.seq_start.data_ptr(),
+                 ctx.seq_slot.data_ptr(), ctx.n_seqs, q.shape[0], heads, int(window or 0), scale, float(cap or 0.0), _ptr(sink),
+                 gp, ldg, 1 if gate_per_head else 0, out_scale, _stream()),
+               "attention_capped_tc", "attention", 2 * q.numel() * q.element_size())
+        return
     if (CAPPED_ATTENTION_MMA and attention_capped_mma_usable(q.dtype, dim, vdim, page_size)
             and getattr(ctx, "cu_seqlens", None) is not None and qp % 16 == 0 and ldq % 8 == 0 and op % 4 == 0
             and ldo % 2 == 0 and (gate_per_head or ((gp or 0) % 4 == 0 and ldg % 2 == 0))):
