@@ -120,6 +120,123 @@ __global__ void __launch_bounds__(128) filter_rope_cache_kernel(
   }
 }
 
+// The same without a filter, for bfloat16 steps of many tokens.  A block owns ROWS_T consecutive tokens of
+// the step and a run of heads: the angles of its tokens are taken once for all its heads, a warp turns a
+// (token, head) at a time with both dims of a pair in one lane, and values pass through shared memory so
+// that a dim's neighbouring positions are written together.
+constexpr int ROWS_T = 16, ROWS_WARPS = 8, VCH = 64;   // tokens a block; warps; value dims a warp turns at a time
+
+template <int NP>     // pairs of dims a lane holds: heads up to 64 * NP wide
+__global__ void __launch_bounds__(ROWS_WARPS * 32) rope_cache_rows_kernel(
+    const bf16* __restrict__ u, long long ldu, const float* __restrict__ inv_freq, int rot, const int* __restrict__ tok_pos,
+    const int* __restrict__ tok_seq, const int* __restrict__ seq_slot, const int* __restrict__ page_table, int table_width,
+    int page_size, bf16* __restrict__ q_out, long long ldq, bf16* __restrict__ kcache, bf16* __restrict__ vcache, int ntok, int H,
+    int G, int D, int Vd, const float* __restrict__ q_norm, const float* __restrict__ k_norm, float norm_eps, float rot_mag,
+    float qt_coef, int qt_every, int v_from_k, int pairs, int unit_after, int heads_a_block, int two) {
+  extern __shared__ float2 turn[];                      // [ROWS_T][rot / 2] (cos, sin)
+  __shared__ int page_of[ROWS_T], off_of[ROWS_T];
+  __shared__ float temper_of[ROWS_T];
+  __shared__ bf16 tile[ROWS_WARPS][ROWS_T][VCH + 2];
+  pdl_release_next();
+  pdl_wait_prior();
+  const int t0 = blockIdx.x * ROWS_T, nt = min(ROWS_T, ntok - t0), half = rot / 2;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x < nt) {
+    const int t = t0 + threadIdx.x, pos = tok_pos[t];
+    page_of[threadIdx.x] = page_table ? page_table[(size_t)seq_slot[tok_seq[t]] * table_width + (pos / page_size) % table_width] : 0;
+    off_of[threadIdx.x] = pos % page_size;
+    temper_of[threadIdx.x] = qt_every > 0 ? 1.0f + qt_coef * logf((float)((pos + 1) / qt_every + 1)) : 1.0f;
+  }
+  for (int e = threadIdx.x; e < nt * half; e += ROWS_WARPS * 32) {
+    float sn, cn;
+    sincosf((float)tok_pos[t0 + e / half] * inv_freq[e % half], &sn, &cn);
+    turn[e] = make_float2(cn * rot_mag, sn * rot_mag);
+  }
+  __syncthreads();
+  const int hb = blockIdx.y * heads_a_block, he = min(H + 2 * G, hb + heads_a_block);
+  // ---- queries and keys
+  const int qk_end = min(he, H + G);
+  for (int w = warp; w < (qk_end - hb) * nt; w += ROWS_WARPS) {
+    const int hh = hb + w / nt, tt = w % nt;
+    if (hh >= H && !kcache) break;
+    const bf16* src = u + (size_t)(t0 + tt) * ldu + (size_t)hh * D;
+    const float* norm_w = hh < H ? q_norm : k_norm;
+    float a[NP], b[NP], ss = 0.f;
+    int da[NP], db[NP];
+#pragma unroll
+    for (int s = 0; s < NP; ++s) {
+      const int p = lane + 32 * s;
+      const bool turns = p < half;
+      da[s] = turns ? (pairs ? 2 * p : p) : rot + 2 * (p - half);
+      db[s] = turns && !pairs ? p + half : da[s] + 1;
+      a[s] = b[s] = 0.f;
+      if (da[s] < D) {
+        if (two && db[s] == da[s] + 1) {                 // D is even here: db < D
+          const float2 v = __bfloat1622float2(*(const __nv_bfloat162*)(src + da[s]));
+          a[s] = v.x;
+          b[s] = v.y;
+        } else {
+          a[s] = to_f32(src[da[s]]);
+          if (db[s] < D) b[s] = to_f32(src[db[s]]);
+        }
+      }
+      ss = fmaf(a[s], a[s], fmaf(b[s], b[s], ss));
+    }
+    if (norm_w) {
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)D + norm_eps);
+#pragma unroll
+      for (int s = 0; s < NP; ++s) {
+        if (da[s] < D) a[s] *= inv * norm_w[da[s]];
+        if (db[s] < D) b[s] *= inv * norm_w[db[s]];
+      }
+    }
+    ss = 0.f;
+#pragma unroll
+    for (int s = 0; s < NP; ++s) {
+      const int p = lane + 32 * s;
+      if (p < half) {
+        const float2 cs = turn[tt * half + p];
+        const float x = a[s] * cs.x - b[s] * cs.y;
+        b[s] = b[s] * cs.x + a[s] * cs.y;
+        a[s] = x;
+      }
+      ss = fmaf(a[s], a[s], fmaf(b[s], b[s], ss));
+    }
+    float factor = hh < H ? temper_of[tt] : 1.0f;
+    if (unit_after) factor *= 1.0f / sqrtf(warp_sum(ss) / (float)D + norm_eps);
+    bf16* dst = hh < H ? q_out + (size_t)(t0 + tt) * ldq + (size_t)hh * D
+                       : kcache + (((size_t)page_of[tt] * G + (hh - H)) * page_size + off_of[tt]) * D;
+#pragma unroll
+    for (int s = 0; s < NP; ++s) {
+      if (da[s] >= D) continue;
+      if (two && db[s] == da[s] + 1) {
+        *(__nv_bfloat162*)(dst + da[s]) = __floats2bfloat162_rn(a[s] * factor, b[s] * factor);
+      } else {
+        dst[da[s]] = from_f32<bf16>(a[s] * factor);
+        if (db[s] < D) dst[db[s]] = from_f32<bf16>(b[s] * factor);
+      }
+    }
+  }
+  // ---- values: rows in, a dim's positions out
+  if (!vcache || he <= H + G) return;
+  const int v_first = max(hb, H + G) - (H + G), v_heads = he - max(hb, H + G), pieces = (Vd + VCH - 1) / VCH;
+  for (int w = warp; w < v_heads * pieces; w += ROWS_WARPS) {
+    const int g = v_first + w / pieces, d0 = (w % pieces) * VCH, nd = min(VCH, Vd - d0);
+    const bf16* src = u + (size_t)t0 * ldu + (v_from_k ? H * D : (H + G) * D) + (size_t)g * Vd + d0;
+    for (int tt = 0; tt < nt; ++tt)
+      for (int d = lane; d < nd; d += 32) tile[warp][tt][d] = src[(size_t)tt * ldu + d];
+    __syncwarp();
+    const int tt = lane % ROWS_T;
+    if (tt < nt) {
+      bf16* dst = vcache + (((size_t)page_of[tt] * G + g) * Vd + d0) * page_size + off_of[tt];
+      for (int d = lane / ROWS_T; d < nd; d += 32 / ROWS_T) dst[(size_t)d * page_size] = tile[warp][tt][d];
+    }
+    __syncwarp();
+  }
+}
+
+constexpr int ROWS_MIN_TOKENS = 64, ROWS_MAX_ROT = 384;   // the angles (8 bytes a pair and token) beside the tiles in 48 KB
+
 // taps: [(H + G) D + G Vd, K] float32 (K = 0: no filter); state: [slots, K - 1, channels] float32.
 // G = 0: the rows hold queries only (a layer that reads another layer's keys and values).
 // q_norm, k_norm: float32 [D] or null (norm_eps is theirs, or unit_after's: not both); v_from_k needs Vd == D.
@@ -136,6 +253,24 @@ GB_EXPORT int gb_filter_rope_cache_ext(const void* u, int dtype, long long ldu, 
   if (v_from_k && (Vd != D || K > 1)) return GB_ERR_SIZE;
   if (unit_after && (q_norm || k_norm)) return GB_ERR_ARG;
   if ((K > 0 && !taps) || (K > 1 && !state) || (rot > 0 && !inv_freq) || qt_every < 0) return GB_ERR_ARG;
+  if (dtype == GB_BF16 && K == 0 && ntok >= ROWS_MIN_TOKENS && rot <= ROWS_MAX_ROT) {
+    // blocks for a few rounds of the SMs: heads are dealt out until there are enough
+    const int tiles = (ntok + ROWS_T - 1) / ROWS_T, all = H + 2 * G;
+    const int runs = min(all, max(1, (4 * 148 + tiles - 1) / tiles)), each = (all + runs - 1) / runs;
+    const int two = D % 2 == 0 && ldu % 2 == 0 && ldq % 2 == 0 && !((uintptr_t)u & 3) && !((uintptr_t)q_out & 3) && !((uintptr_t)kcache & 3);
+    const size_t smem = (size_t)ROWS_T * (rot / 2) * sizeof(float2);
+#define ROWS(NP)                                                                                                               \
+  gb_launch(rope_cache_rows_kernel<NP>, dim3(tiles, (all + each - 1) / each), dim3(ROWS_WARPS * 32), smem, stream, (const bf16*)u, \
+            ldu, inv_freq, rot, tok_pos, tok_seq, seq_slot, page_table, table_width, page_size, (bf16*)q_out, ldq, (bf16*)kcache,  \
+            (bf16*)vcache, ntok, H, G, D, Vd, q_norm, k_norm, norm_eps, rot_mag, qt_coef, qt_every, v_from_k, pairs, unit_after, \
+            each, two)
+    if (D <= 64) ROWS(1);
+    else if (D <= 128) ROWS(2);
+    else if (D <= 256) ROWS(4);
+    else ROWS(8);
+#undef ROWS
+    return gb_launch_status();
+  }
   const dim3 grid(ntok, H + 2 * G);
   if (dtype == GB_F32)
     gb_launch(filter_rope_cache_kernel<float>, grid, 128, 0, stream, (const float*)u, ldu, taps, state, K, inv_freq, rot,

@@ -221,9 +221,37 @@ attention_capped_mma_kernel(const bf16* __restrict__ q, long long q_stride, bf16
 // A step of single tokens.  The 16 rows of an MMA are the query heads that share a kv head (in
 // chunks of 16), all at the sequence's one new position, so a key or value is read once for all
 // of them; the SPLIT warps of a CTA take every SPLIT-th block of 32 keys each, and their parts
-// (maximum, sum, weighted values per row) meet in shared memory, added in warp order.
-// grid (sequences, kv heads * chunks of 16 heads); block SPLIT * 32.
-__global__ void __launch_bounds__(SPLIT * 32)
+// (maximum, sum, weighted values per row) meet in shared memory, added in warp order.  A step with
+// few sequences deals a head's blocks to the CTAs of a cluster (up to MAX_SPREAD) as well: each adds its
+// own warps' parts first, then every CTA adds the cluster's parts, in the order of the ranks, for its
+// share of the results.
+// grid (sequences, kv heads * chunks of 16 heads, CTAs of a cluster); block SPLIT * 32.
+constexpr int MAX_SPREAD = 8;
+
+__device__ __forceinline__ uint32_t spread_rank() {
+  uint32_t r;
+  asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
+  return r;
+}
+__device__ __forceinline__ uint32_t spread_size() {
+  uint32_t r;
+  asm volatile("mov.u32 %0, %%cluster_nctarank;" : "=r"(r));
+  return r;
+}
+__device__ __forceinline__ void spread_sync() {
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// The float at this place of the shared memory of the cluster's CTA `rank`.
+__device__ __forceinline__ float ld_peer(const float* local, uint32_t rank) {
+  uint32_t addr;
+  float v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(addr) : "r"((uint32_t)__cvta_generic_to_shared(local)), "r"(rank));
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+  return v;
+}
+
+__global__ void __launch_bounds__(SPLIT * 32, 1)
 attention_capped_single_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __restrict__ out, long long out_stride,
                          const bf16* __restrict__ kcache, const bf16* __restrict__ vcache, PagedKV kv,
                          const int* __restrict__ cu_seqlens, const int* __restrict__ seq_start,
@@ -277,7 +305,8 @@ attention_capped_single_kernel(const bf16* __restrict__ q, long long q_stride, b
   const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f, cap2 = cap * LOG2E, scale2 = scale * LOG2E;
   const int win_blk = lo_first / KEYS, kept_blks = min((keep_first + KEYS - 1) / KEYS, win_blk);
   const int n_blks = kept_blks + last / KEYS - win_blk + 1;
-  for (int it = warp; it < n_blks; it += SPLIT) {
+  const int rank = (int)spread_rank(), spread = (int)spread_size();
+  for (int it = warp + rank * SPLIT; it < n_blks; it += SPLIT * spread) {
     const int key0 = (it < kept_blks ? it : win_blk + it - kept_blks) * KEYS;
     const int page = kv.page_table[(size_t)slot * kv.table_width + (key0 / kv.page_size) % kv.table_width];
     const size_t page_base = ((size_t)page * kv.num_kv_heads + kvh) * kv.page_size * HD;
@@ -342,10 +371,12 @@ attention_capped_single_kernel(const bf16* __restrict__ q, long long q_stride, b
   }
   l0 = quad_sum(l0);
   l1 = quad_sum(l1);
-  extern __shared__ float parts[];            // [SPLIT][16] maxima, [SPLIT][16] sums, [SPLIT][16][VD] weighted values
+  extern __shared__ float parts[];            // [SPLIT][16] maxima, [SPLIT][16] sums, [SPLIT][16][VD] weighted values, the CTA's [16] and [16]
   float* pm = parts;
   float* pl = pm + SPLIT * 16;
   float* po = pl + SPLIT * 16;
+  float* cm = po + SPLIT * 16 * VD;
+  float* cl = cm + 16;
   if (c == 0) {
     pm[warp * 16 + g] = m0; pl[warp * 16 + g] = l0;
     pm[warp * 16 + g + 8] = m1; pl[warp * 16 + g + 8] = l1;
@@ -356,6 +387,49 @@ attention_capped_single_kernel(const bf16* __restrict__ q, long long q_stride, b
     *(float2*)(po + (size_t)(warp * 16 + g + 8) * VD + d * 8 + 2 * c) = make_float2(o[d][2], o[d][3]);
   }
   __syncthreads();
+  if (spread > 1) {
+    // the CTA's own parts become one, in the first warp's place (a thread reads and writes its own element)
+    for (int idx = threadIdx.x; idx < rows * VD; idx += SPLIT * 32) {
+      const int row = idx / VD, col = idx - row * VD;
+      float top = -INFINITY, total = 0.f, acc = 0.f;
+#pragma unroll
+      for (int w = 0; w < SPLIT; ++w) top = fmaxf(top, pm[w * 16 + row]);
+#pragma unroll
+      for (int w = 0; w < SPLIT; ++w) {
+        const float m = pm[w * 16 + row];
+        const float wt = m == -INFINITY ? 0.f : exp2f(m - top);
+        total = fmaf(wt, pl[w * 16 + row], total);
+        acc = fmaf(wt, po[(size_t)(w * 16 + row) * VD + col], acc);
+      }
+      po[(size_t)row * VD + col] = acc;
+      if (col == 0) { cm[row] = top; cl[row] = total; }
+    }
+    spread_sync();
+    for (int idx = threadIdx.x + rank * SPLIT * 32; idx < rows * VD; idx += SPLIT * 32 * spread) {
+      const int row = idx / VD, col = idx - row * VD;
+      const float s2 = sink ? sink[head_base + row] * LOG2E : -INFINITY;
+      float ms[MAX_SPREAD], top = s2;
+#pragma unroll
+      for (int r = 0; r < MAX_SPREAD; ++r) {
+        ms[r] = r < spread ? ld_peer(cm + row, r) : -INFINITY;
+        top = fmaxf(top, ms[r]);
+      }
+      float total = sink ? exp2f(s2 - top) : 0.f, acc = 0.f;
+#pragma unroll
+      for (int r = 0; r < MAX_SPREAD; ++r) {
+        if (r >= spread) break;
+        const float wt = ms[r] == -INFINITY ? 0.f : exp2f(ms[r] - top);
+        total = fmaf(wt, ld_peer(cl + row, r), total);
+        acc = fmaf(wt, ld_peer(po + (size_t)row * VD + col, r), acc);
+      }
+      float a = acc * out_scale / total;
+      const size_t at = (size_t)(head_base + row) * VD + col;
+      if (gate) a *= 1.0f / (1.0f + __expf(-__bfloat162float(gate[(size_t)tok0 * gate_stride + (gate_per_head ? head_base + row : at)])));
+      out[(size_t)tok0 * out_stride + at] = __float2bfloat16_rn(a);
+    }
+    spread_sync();                             // no CTA leaves while another still reads its parts
+    return;
+  }
   for (int idx = threadIdx.x; idx < rows * VD; idx += SPLIT * 32) {
     const int row = idx / VD, col = idx - row * VD;
     const float s2 = sink ? sink[head_base + row] * LOG2E : -INFINITY;
@@ -401,13 +475,13 @@ GB_EXPORT int gb_attention_capped_mma(const void* q, long long q_stride, void* o
   if (single) {
     // every sequence brings one token (ntok == n_seqs)
     if (ntok != n_seqs) return GB_ERR_ARG;
-    const size_t smem = (size_t)SPLIT * 16 * (VD + 2) * sizeof(float);
+    const size_t smem = ((size_t)SPLIT * 16 * (VD + 2) + 32) * sizeof(float);
     static bool raised = false;
     if (!raised) {
       cudaFuncSetAttribute(attention_capped_single_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       raised = true;
     }
-    const dim3 sgrid(n_seqs, nkv * ((rep + 15) / 16));
+    dim3 sgrid(n_seqs, nkv * ((rep + 15) / 16));
     if ((size_t)sgrid.x * sgrid.y > 2 * 148) {
       gb_launch(attention_capped_single_kernel, sgrid, SPLIT * 32, smem, stream,
           (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kcache, (const bf16*)vcache, kv, cu_seqlens,
@@ -415,7 +489,18 @@ GB_EXPORT int gb_attention_capped_mma(const void* q, long long q_stride, void* o
     } else {
       // few CTAs: started only when the kernel before has ended, so that they spread one to an SM instead of
       // sharing the few SMs that had room while that kernel ran
+      // and, where SMs are left over, a head's keys are dealt to the CTAs of a cluster (one CTA fits an SM)
+      int spread = 1;
+      while (spread < MAX_SPREAD && (size_t)sgrid.x * sgrid.y * spread * 2 <= 148) spread *= 2;
+      sgrid.z = spread;
       cudaLaunchConfig_t cfg = {};
+      cudaLaunchAttribute attr[1];
+      attr[0].id = cudaLaunchAttributeClusterDimension;
+      attr[0].val.clusterDim.x = 1;
+      attr[0].val.clusterDim.y = 1;
+      attr[0].val.clusterDim.z = spread;
+      cfg.attrs = attr;
+      cfg.numAttrs = spread > 1 ? 1 : 0;
       cfg.gridDim = sgrid;
       cfg.blockDim = dim3(SPLIT * 32);
       cfg.dynamicSmemBytes = smem;
