@@ -450,7 +450,7 @@ FEZOZEN_B = {
          "mlp": _fezozen_moe(8, 3, 64)},
         {"type": "attention", "mixer": _FB_CAPPED, "mlp": _fezozen_moe(6, 1, 96)},
         {"type": "attention_2", "mixer": _fezozen_unit(6, 2, 32, 64, 0.25, 65, _fezozen_rot(1e4, 32)), "mlp": _fezozen_moe(8, 3, 64)},
-        {"type": "latent_attention", "mixer": _fezozen_latent(4, 32, 32, 64, 64, 0.125, 64, 1e4), "mlp": _fezozen_moe(6, 2, 72)},
+        {"type": "latent_attention", "mixer": _fezozen_latent(5, 32, 32, 64, 64, 0.14, 64, 1e4), "mlp": _fezozen_moe(6, 2, 72)},
         {"type": "attention", "mixer": _FB_CAPPED, "mlp": _fezozen_moe(6, 1, 96), "weights_of": 1},
     ],
 }
